@@ -10,6 +10,7 @@ from .base import (
 )
 from .qwen3 import PRESETS, Qwen3Config
 from .qwen3 import preset as _qwen3_preset
+from .fimilix import FIMILIX_PRESETS, FimilixConfig
 from .kirenex import KIRENEX_PRESETS, KirenexConfig
 from .limazen import LIMAZEN_PRESETS, LimazenConfig
 from .topidra import TOPIDRA_PRESETS, TopidraConfig
@@ -18,6 +19,8 @@ from .vopozen import VOPOZEN_PRESETS, VopozenConfig
 
 def preset(name: str, **overrides):
     """The configuration of a named shape, of whichever architecture has that name."""
+    if name in FIMILIX_PRESETS:
+        return FimilixConfig(**{**FIMILIX_PRESETS[name], **overrides})
     if name in VOPOZEN_PRESETS:
         return VopozenConfig(**{**VOPOZEN_PRESETS[name], **overrides})
     if name in KIRENEX_PRESETS:
@@ -27,12 +30,12 @@ def preset(name: str, **overrides):
     if name in TOPIDRA_PRESETS:
         return TopidraConfig(**{**TOPIDRA_PRESETS[name], **overrides})
     if name not in PRESETS:
-        raise ValueError(f"unknown preset {name!r}; known: {sorted(PRESETS) + sorted(TOPIDRA_PRESETS) + sorted(LIMAZEN_PRESETS) + sorted(KIRENEX_PRESETS) + sorted(VOPOZEN_PRESETS)}")
+        raise ValueError(f"unknown preset {name!r}; known: {sorted(PRESETS) + sorted(TOPIDRA_PRESETS) + sorted(LIMAZEN_PRESETS) + sorted(KIRENEX_PRESETS) + sorted(VOPOZEN_PRESETS) + sorted(FIMILIX_PRESETS)}")
     return _qwen3_preset(name, **overrides)
 
 
 __all__ = [
     "DTYPE_BYTES", "Architecture", "load_config", "read_config_json", "register_architecture",
     "resolve_architecture", "supported_architectures", "unregister_architecture",
-    "PRESETS", "Qwen3Config", "preset", "TOPIDRA_PRESETS", "TopidraConfig", "LIMAZEN_PRESETS", "LimazenConfig", "KIRENEX_PRESETS", "KirenexConfig", "VOPOZEN_PRESETS", "VopozenConfig",
+    "PRESETS", "Qwen3Config", "preset", "TOPIDRA_PRESETS", "TopidraConfig", "LIMAZEN_PRESETS", "LimazenConfig", "KIRENEX_PRESETS", "KirenexConfig", "VOPOZEN_PRESETS", "VopozenConfig", "FIMILIX_PRESETS", "FimilixConfig",
 ]

@@ -18,6 +18,10 @@
 //            (max, sum, unnormalised output) to scratch memory and the block that arrives last at
 //            the (sequence, KV head) counter merges the splits in order and resets the counter.
 //
+// A soft cap on the scores (cap * tanh(score / cap), before the mask) and a factor on the outputs are
+// parameters of the variants with sinks, gates and split weights; a token's output row may be part of a
+// wider row (`out_stride`).
+//
 // Keys outside [first visible key, context length) are loaded as zeros and masked by replacing
 // their scores, so stale or non-finite page contents cannot reach a result. Head sizes are
 // multiples of 16 up to 256 (a runtime value under a compile-time bound of 128 or 256).
@@ -151,12 +155,14 @@ __device__ __forceinline__ void ldmatrix_x4_trans_at(uint32_t (&r)[4], uint32_t 
 // tile that every row sees completely. Scores stay unscaled; the scale enters the exponent.
 // SPLIT: a weight enters the second product as the sum of two bfloat16 numbers (its rounded value and
 // the rounded rest), each multiplied exactly and added in 32-bit: the weights keep 16 bits of
-// mantissa instead of 8, at one more MMA per step of P V.
+// mantissa instead of 8, at one more MMA per step of P V. With `cap_in` != 0 (SPLIT only) a score s becomes
+// cap_out * tanh(cap_in s / (2 log2 e)) = cap_out - 2 cap_out / (1 + 2^(cap_in s)), already in the exponent's
+// base-2 units (c = 1): the absolute error is about cap_out times a float's rounding, whatever the score.
 template <int MAX_DIM, bool EXACT, int PAIRS, bool UPPER, bool SPLIT = false>
 __device__ __forceinline__ void warp_tile(const uint32_t (&qf)[MAX_DIM / 16][4], uint32_t k_addr, uint32_t v_addr,
                                           int dim, float (&o)[MAX_DIM / 8][4], float (&m_run)[2], float (&l_run)[2],
                                           bool masked, int key0, int p0, int p1, int key_lo, int window, float c,
-                                          int t, int keep = 0) {
+                                          int t, int keep = 0, float cap_in = 0.f, float cap_out = 0.f) {
   constexpr int KSTEPS = MAX_DIM / 16, NT_O = MAX_DIM / 8, NT_S = PAIRS * 2;
   const int dk = EXACT ? KSTEPS : (dim >> 4);
   const uint32_t row_bytes = (uint32_t)((EXACT ? MAX_DIM : dim) + PAD) * 2;
@@ -197,6 +203,16 @@ __device__ __forceinline__ void warp_tile(const uint32_t (&qf)[MAX_DIM / 16][4],
             mma_bf16(s[2 * n2 + 1], qf[k0 + u], b[u][2], b[u][3]);
           }
         }
+      }
+    }
+  }
+  if (SPLIT && cap_in != 0.f) {
+#pragma unroll
+    for (int n = 0; n < NT_S; ++n) {
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        if (!UPPER && e >= 2) continue;
+        s[n][e] = cap_out - __fdividef(2.f * cap_out, 1.f + fast_exp2(s[n][e] * cap_in));
       }
     }
   }
@@ -284,8 +300,9 @@ __device__ __forceinline__ void warp_tile(const uint32_t (&qf)[MAX_DIM / 16][4],
 
 // ------------------------------------------------------------------------------- prefill
 // SINK: the variant for attention with a sink per head (`sinks`, natural-log units: it joins the
-// denominator only), a 32-bit gate per (token, head) on the output (`gates`), either may be null, and
-// weights that keep 16 bits of mantissa in the second product (SPLIT above).
+// denominator only), a 32-bit gate per (token, head) on the output (`gates`), either may be null, a soft cap on the
+// scores (see warp_tile), a factor on every output (`out_scale`), and weights that keep 16 bits of mantissa in the
+// second product (SPLIT above).
 template <int MAX_DIM, bool EXACT, bool SINK = false>
 __global__ void __launch_bounds__(THREADS)
 attention_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_pool, const bf16* __restrict__ v_pool,
@@ -293,7 +310,8 @@ attention_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_
                          const int* __restrict__ cu_q, const int* __restrict__ ctx_len,
                          const int* __restrict__ tile_seq, const int* __restrict__ tile_q0, int q_heads, int kv_heads,
                          int dim_arg, int page_tokens, float scale_log2, int window, int chunk_shift, int page_shift,
-                         const float* __restrict__ sinks, const float* __restrict__ gates, int keep_first) {
+                         const float* __restrict__ sinks, const float* __restrict__ gates, int keep_first, float cap_in,
+                         float cap_out, float out_scale, long out_stride) {
   constexpr int KSTEPS = MAX_DIM / 16, NT_O = MAX_DIM / 8;
   extern __shared__ __align__(16) uint8_t smem_raw[];
   const int dim = EXACT ? MAX_DIM : dim_arg;
@@ -376,7 +394,7 @@ attention_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_
       const bool masked = tile * BKEYS + BKEYS - 1 > p_warp || tile * BKEYS < key_lo || window != 0;
       warp_tile<MAX_DIM, EXACT, BKEYS / 16, true, SINK>(qf, k_base + buf * buf_bytes, v_base + buf * buf_bytes, dim, o, m_run,
                                                         l_run, masked, tile * BKEYS, p0, p1, key_lo, window, scale_log2, t,
-                                                        keep_first);
+                                                        keep_first, cap_in, cap_out);
     }
     __syncthreads();   // the buffer may be overwritten by the next iteration's prefetch
   }
@@ -395,8 +413,9 @@ attention_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_
       // the row's maximum is finite (a query sees itself); scores are unscaled, the sink is not to be scaled
       if (sinks) inv = 1.0f / (l_run[r] + fast_exp2(sinks[head] * 1.4426950408889634f - m_run[r] * scale_log2));
       if (gates) inv *= gates[(size_t)(row0 + q0 + row) * q_heads + head];
+      inv *= out_scale;
     }
-    bf16* dst = out + ((size_t)(row0 + q0 + row) * q_heads + head) * dim;
+    bf16* dst = out + (size_t)(row0 + q0 + row) * out_stride + head * dim;
 #pragma unroll
     for (int n = 0; n < NT_O; ++n) {
       if (EXACT || n * 8 < dim)
@@ -427,7 +446,8 @@ attention_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_p
                         const int* __restrict__ seq_list, int q_heads, int kv_heads, int dim_arg, int page_tokens,
                         float scale_log2, int window, int splits, float* __restrict__ partials,
                         unsigned* __restrict__ counters, int chunk_shift, int page_shift,
-                        const float* __restrict__ sinks, const float* __restrict__ gates, int keep_first, int kv_share) {
+                        const float* __restrict__ sinks, const float* __restrict__ gates, int keep_first, int kv_share,
+                        float cap_in, float cap_out, float out_scale, long out_stride) {
   constexpr int KSTEPS = MAX_DIM / 16, NT_O = MAX_DIM / 8;
   extern __shared__ __align__(16) uint8_t smem_raw[];
   const int dim = EXACT ? MAX_DIM : dim_arg;
@@ -526,7 +546,8 @@ attention_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_p
     // only the tile that holds the last key, or the first visible one, needs the comparisons
     const bool masked = tile * BKEYS + BKEYS - 1 > p || tile * BKEYS < key_lo;
     warp_tile<MAX_DIM, EXACT, 1, UPPER, SINK>(qf, k_base + buf * buf_bytes, v_base + buf * buf_bytes, dim, o, m_run, l_run,
-                                              masked, tile * BKEYS + warp * 16, p, p, key_lo, 0, scale_log2, t, keep);
+                                              masked, tile * BKEYS + warp * 16, p, p, key_lo, 0, scale_log2, t, keep, cap_in,
+                                              cap_out);
     __syncthreads();
   }
   cp_async_wait<0>();
@@ -557,6 +578,7 @@ attention_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_p
     if (SINK && sinks) l_all += fast_exp2(sinks[head0 + r] * 1.4426950408889634f - base * c);
     float value = l_all > 0.f ? acc / l_all : 0.f;
     if (SINK && gates) value *= gates[(size_t)row * q_heads + head0 + r];
+    if (SINK) value *= out_scale;
     return value;
   };
   if (CLUSTER) {
@@ -602,7 +624,7 @@ attention_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_p
         acc += recv_acc[(size_t)s2 * per + k] * f;
         l_all += recv_ml[((size_t)s2 * group + r) * 2 + 1] * f;
       }
-      out[((size_t)row * q_heads + head0 + r) * dim + col] = __float2bfloat16_rn(finish(acc, l_all, base, r));
+      out[(size_t)row * out_stride + (head0 + r) * dim + col] = __float2bfloat16_rn(finish(acc, l_all, base, r));
     }
     return;
   }
@@ -623,7 +645,7 @@ attention_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_p
       l_all += src[dim + 1] * f;
     }
     if (splits == 1) {
-      out[((size_t)row * q_heads + head0 + r) * dim + col] = __float2bfloat16_rn(finish(acc, l_all, base, r));
+      out[(size_t)row * out_stride + (head0 + r) * dim + col] = __float2bfloat16_rn(finish(acc, l_all, base, r));
     } else {
       my_partial[r * mstride + col] = acc;
       if (col == 0) { my_partial[r * mstride + dim] = m_all; my_partial[r * mstride + dim + 1] = l_all; }
@@ -686,7 +708,8 @@ attention_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_p
       if (i0 + e * THREADS >= group * dim) break;
       float value = l_total[r[e]] > 0.f ? acc[e] / l_total[r[e]] : 0.f;
       if (SINK && gates) value *= gates[(size_t)row * q_heads + head0 + r[e]];
-      out[((size_t)row * q_heads + head0 + r[e]) * dim + col[e]] = __float2bfloat16_rn(value);
+      if (SINK) value *= out_scale;
+      out[(size_t)row * out_stride + (head0 + r[e]) * dim + col[e]] = __float2bfloat16_rn(value);
     }
   }
   if (threadIdx.x == 0) counters[tile_id] = 0;
@@ -778,25 +801,39 @@ int launch_decode_cluster(int group, dim3 grid, size_t smem, cudaStream_t stream
 }
 }  // namespace
 
-// Prompt portions (any number of queries per sequence), listed as tiles of 64 queries.
+namespace {
+// How the kernels take a scale and a soft cap (0: none): with a cap the scores leave the cap in base-2 units.
+struct ScoreUnits { float scale_log2, cap_in, cap_out; };
+ScoreUnits score_units(float scale, float softcap) {
+  const double log2e = 1.4426950408889634;
+  if (softcap > 0.f) return {1.f, (float)(2.0 * log2e * scale / softcap), (float)(log2e * softcap)};
+  return {scale * 1.4426950408889634f, 0.f, 0.f};
+}
+}  // namespace
+
+// Prompt portions (any number of queries per sequence), listed as tiles of 64 queries. softcap > 0: every score becomes
+// softcap * tanh(score / softcap); out_scale multiplies every output; out_stride: elements from a token's output row to the next.
 LB_EXPORT int lb_attention_prefill_bf16(const void* q, const void* k_pool, const void* v_pool, void* out,
                                         const int* block_table, int table_width, const int* cu_q, const int* ctx_len,
                                         const int* tile_seq, const int* tile_q0, int n_tiles, int q_heads, int kv_heads,
                                         int dim, int page_tokens, float scale, int window, const float* sinks,
-                                        const float* gates, int exact_weights, int keep_first, cudaStream_t stream) {
+                                        const float* gates, int exact_weights, int keep_first, float softcap, float out_scale,
+                                        long out_stride, cudaStream_t stream) {
   if (n_tiles <= 0) return 0;
   if (dim <= 0 || dim % 16 || dim > 256 || kv_heads <= 0 || q_heads % kv_heads || q_heads > 65535) return LB_ERR_SIZE;
   if (keep_first < 0 || (keep_first > 0 && window <= 0)) return LB_ERR_SIZE;
-  const bool sink = sinks || gates || exact_weights;
+  if (out_stride < (long)q_heads * dim || out_stride % 2 || !(softcap >= 0.f)) return LB_ERR_SIZE;
+  const bool sink = sinks || gates || exact_weights || softcap > 0.f || out_scale != 1.f;
   configure_once();
   const size_t smem = prefill_smem(dim, k_pool == v_pool);
-  const float scale_log2 = scale * 1.4426950408889634f;
+  const ScoreUnits u = score_units(scale, softcap);
+  const float scale_log2 = u.scale_log2;
   const int chunk_shift = (dim >> 3) <= THREADS ? exact_log2(dim >> 3) : -1, page_shift = exact_log2(page_tokens);
   dim3 grid(n_tiles, q_heads), block(THREADS);
   int code;
 #define LB_PREFILL_ARGS (const bf16*)q, (const bf16*)k_pool, (const bf16*)v_pool, (bf16*)out, block_table, table_width, cu_q, \
                         ctx_len, tile_seq, tile_q0, q_heads, kv_heads, dim, page_tokens, scale_log2, window, chunk_shift, page_shift, \
-                        sinks, gates, keep_first
+                        sinks, gates, keep_first, u.cap_in, u.cap_out, out_scale, out_stride
   if (sink) {
     if (dim == 128) code = lb_launch(attention_prefill_kernel<128, true, true>, grid, block, smem, stream, LB_PREFILL_ARGS);
     else if (dim < 128) code = lb_launch(attention_prefill_kernel<128, false, true>, grid, block, smem, stream, LB_PREFILL_ARGS);
@@ -827,7 +864,7 @@ LB_EXPORT int lb_attention_decode_bf16(const void* q, const void* k_pool, const 
                                        int page_tokens, float scale, int window, int splits, float* partials,
                                        long partial_floats, unsigned* counters, int n_counters, int stages,
                                        const float* sinks, const float* gates, int exact_weights, int keep_first,
-                                       int kv_share, cudaStream_t stream) {
+                                       int kv_share, float softcap, float out_scale, long out_stride, cudaStream_t stream) {
   if (n_seqs <= 0) return 0;
   if (keep_first < 0 || (keep_first > 0 && window <= 0) || kv_share < 1 || kv_heads % kv_share) return LB_ERR_SIZE;
   if (dim <= 0 || dim % 16 || dim > 256 || kv_heads <= 0 || q_heads % kv_heads || q_heads / kv_heads > 16 ||
@@ -838,11 +875,13 @@ LB_EXPORT int lb_attention_decode_bf16(const void* q, const void* k_pool, const 
     return LB_ERR_SIZE;
   configure_once();
   // two K/V stages (three blocks an SM) exist for the served head size with at most 8 heads per KV head
-  const bool sink = sinks || gates || exact_weights;
+  if (out_stride < (long)q_heads * dim || !(softcap >= 0.f)) return LB_ERR_SIZE;
+  const bool sink = sinks || gates || exact_weights || softcap > 0.f || out_scale != 1.f;
   const bool two_stages = !sink && stages == 2 && dim == 128 && q_heads / kv_heads <= 8;
   const size_t smem = decode_smem(dim, two_stages ? 2 : 3, k_pool == v_pool);
   if ((3 * (size_t)splits + 1) * (q_heads / kv_heads) * sizeof(float) > smem) return LB_ERR_SIZE;   // merge factors
-  const float scale_log2 = scale * 1.4426950408889634f;
+  const ScoreUnits u = score_units(scale, softcap);
+  const float scale_log2 = u.scale_log2;
   const int chunk_shift = (dim >> 3) <= THREADS ? exact_log2(dim >> 3) : -1, page_shift = exact_log2(page_tokens);
   dim3 grid(n_seqs, kv_heads, splits);
   int code;
@@ -850,27 +889,28 @@ LB_EXPORT int lb_attention_decode_bf16(const void* q, const void* k_pool, const 
   if (sink) {
     code = launch_decode_sink(dim, grid, smem, stream, (const bf16*)q, (const bf16*)k_pool, (const bf16*)v_pool, (bf16*)out,
                               block_table, table_width, cu_q, ctx_len, seq_list, q_heads, kv_heads, dim, page_tokens,
-                              scale_log2, window, splits, partials, counters, chunk_shift, page_shift, sinks, gates, keep_first, kv_share);
+                              scale_log2, window, splits, partials, counters, chunk_shift, page_shift, sinks, gates, keep_first, kv_share, u.cap_in, u.cap_out,
+                              out_scale, out_stride);
   } else if (two_stages) {
     if (decode_cluster_fits(dim, q_heads / kv_heads, splits, smem))
       code = lb_launch_cluster(attention_decode_kernel<128, true, false, true, 2>, grid, dim3(THREADS), smem, stream, grid.z,
                                (const bf16*)q, (const bf16*)k_pool, (const bf16*)v_pool, (bf16*)out, block_table, table_width,
                                cu_q, ctx_len, seq_list, q_heads, kv_heads, dim, page_tokens, scale_log2, window, splits,
-                               (float*)nullptr, (unsigned*)nullptr, chunk_shift, page_shift, no_floats, no_floats, keep_first, kv_share);
+                               (float*)nullptr, (unsigned*)nullptr, chunk_shift, page_shift, no_floats, no_floats, keep_first, kv_share, 0.f, 0.f, 1.f, out_stride);
     else
       code = lb_launch(attention_decode_kernel<128, true, false, false, 2>, grid, dim3(THREADS), smem, stream, (const bf16*)q,
                        (const bf16*)k_pool, (const bf16*)v_pool, (bf16*)out, block_table, table_width, cu_q, ctx_len, seq_list,
                        q_heads, kv_heads, dim, page_tokens, scale_log2, window, splits, partials, counters, chunk_shift,
-                       page_shift, no_floats, no_floats, keep_first, kv_share);
+                       page_shift, no_floats, no_floats, keep_first, kv_share, 0.f, 0.f, 1.f, out_stride);
   } else if (decode_cluster_fits(dim, q_heads / kv_heads, splits, smem))
     code = launch_decode_cluster(q_heads / kv_heads, grid, smem, stream, (const bf16*)q, (const bf16*)k_pool,
                                  (const bf16*)v_pool, (bf16*)out, block_table, table_width, cu_q, ctx_len, seq_list,
                                  q_heads, kv_heads, dim, page_tokens, scale_log2, window, splits, (float*)nullptr,
-                                 (unsigned*)nullptr, chunk_shift, page_shift, no_floats, no_floats, keep_first, kv_share);
+                                 (unsigned*)nullptr, chunk_shift, page_shift, no_floats, no_floats, keep_first, kv_share, 0.f, 0.f, 1.f, out_stride);
   else
     code = launch_decode(dim, q_heads / kv_heads, grid, smem, stream, (const bf16*)q, (const bf16*)k_pool,
                          (const bf16*)v_pool, (bf16*)out, block_table, table_width, cu_q, ctx_len, seq_list,
                          q_heads, kv_heads, dim, page_tokens, scale_log2, window, splits, partials, counters,
-                         chunk_shift, page_shift, no_floats, no_floats, keep_first, kv_share);
+                         chunk_shift, page_shift, no_floats, no_floats, keep_first, kv_share, 0.f, 0.f, 1.f, out_stride);
   return code ? code : lb_last_error();
 }

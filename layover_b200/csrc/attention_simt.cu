@@ -11,7 +11,8 @@
 // pointer or an equal size: values of another size than keys (`vdim`, out is [T, q_heads * vdim]);
 // a learned sink per query head, a score without key or value that only enlarges the softmax's
 // denominator, o = sum_j exp(s_j) V_j / (exp(sink_h) + sum_j exp(s_j)); and a gate per (token,
-// head), a 32-bit factor on the head's output. Keys are walked in tiles of 32 aligned to absolute
+// head), a 32-bit factor on the head's output. Two more: a soft cap, s_j <- cap * tanh(s_j / cap), and a factor
+// `out_scale` on every output. Keys are walked in tiles of 32 aligned to absolute
 // positions (tile i holds keys [32 i, 32 i + 32)), each score is one sequential dot product and
 // the running maximum / sum follow the same recurrence for every row, so a row's result does
 // not depend on how the tokens were cut into steps or on which other rows share its block.
@@ -54,7 +55,7 @@ paged_attention_simt_kernel(const T* __restrict__ q, const T* __restrict__ k_poo
                             const int* __restrict__ tile_seq, const int* __restrict__ tile_q0, int q_heads,
                             int kv_heads, int dim, int page_tokens, float scale, int window, int vdim,
                             const float* __restrict__ sinks, const float* __restrict__ gates, int mask_chunk,
-                            int keep_first) {
+                            int keep_first, float cap, float out_scale, long out_stride) {
   extern __shared__ __align__(16) float smem[];
   pdl_launch_dependents();
   pdl_wait();
@@ -131,7 +132,9 @@ paged_attention_simt_kernel(const T* __restrict__ q, const T* __restrict__ k_poo
       const float* qr = q_s + row * dim;
       const float* kr = k_s + lane * (dim + 1);
       for (int c = 0; c < dim; ++c) s = fmaf(qr[c], kr[c], s);
-      s = seen ? s * scale : -INFINITY;
+      s *= scale;
+      if (cap > 0.f) s = cap * tanhf(s / cap);
+      s = seen ? s : -INFINITY;
       const float tile_max = warp_max(s);
       if (tile_max == -INFINITY) continue;  // nothing of this tile is seen by this row
       const float m_new = fmaxf(m[r], tile_max);
@@ -155,7 +158,7 @@ paged_attention_simt_kernel(const T* __restrict__ q, const T* __restrict__ k_poo
   for (int r = 0; r < ROWS_PER_WARP; ++r) {
     const int row = warp * ROWS_PER_WARP + r;
     if (row >= n_q) continue;
-    T* o = out + ((size_t)(row0 + q0 + row) * q_heads + head) * vdim;
+    T* o = out + (size_t)(row0 + q0 + row) * out_stride + head * vdim;
     float denominator = l[r], keep = 1.f;
     if (sinks) {                                   // the sink joins the denominator only; m is finite (a row sees itself)
       const float sink = sinks[head], top = fmaxf(m[r], sink);
@@ -169,6 +172,7 @@ paged_attention_simt_kernel(const T* __restrict__ q, const T* __restrict__ k_poo
       if (d < vdim) {
         float value = sinks ? acc[r][c] * keep / denominator : acc[r][c] / l[r];
         if (gates) value *= gate;
+        value *= out_scale;
         Elem<T>::store(o + d, value);
       }
     }
@@ -182,10 +186,12 @@ LB_EXPORT int lb_attention_simt(int dtype, const void* q, const void* k_pool, co
                                 const int* block_table, int table_width, const int* cu_q, const int* ctx_len,
                                 const int* tile_seq, const int* tile_q0, int n_tiles, int q_heads, int kv_heads,
                                 int dim, int page_tokens, float scale, int window, int vdim, const float* sinks,
-                                const float* gates, int mask_chunk, int keep_first, cudaStream_t stream) {
+                                const float* gates, int mask_chunk, int keep_first, float softcap, float out_scale,
+                                long out_stride, cudaStream_t stream) {
   if (n_tiles <= 0) return 0;
   if (dim <= 0 || dim > MAX_DIM || dim % 4 || kv_heads <= 0 || q_heads % kv_heads || q_heads > 65535) return LB_ERR_SIZE;
   if (vdim <= 0 || vdim > MAX_DIM || vdim % 4 || keep_first < 0 || (keep_first && mask_chunk)) return LB_ERR_SIZE;
+  if (!(softcap >= 0.f) || out_stride < (long)q_heads * vdim) return LB_ERR_SIZE;
   // q rows, key rows padded by one float, value rows (16-byte aligned: both sizes are multiples of 4)
   const size_t smem = (size_t)(BQ * dim + BKEYS * (dim + 1) + BKEYS * vdim) * sizeof(float);
   dim3 grid(n_tiles, q_heads);
@@ -196,7 +202,7 @@ LB_EXPORT int lb_attention_simt(int dtype, const void* q, const void* k_pool, co
       cudaFuncSetAttribute(paged_attention_simt_kernel<T, ACC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);     \
     lb_launch(paged_attention_simt_kernel<T, ACC>, grid, WARPS * 32, smem, stream, (const T*)q, (const T*)k_pool,            \
               (const T*)v_pool, (T*)out, block_table, table_width, cu_q, ctx_len, tile_seq, tile_q0, q_heads, kv_heads, dim, \
-              page_tokens, scale, window, vdim, sinks, gates, mask_chunk, keep_first);                                       \
+              page_tokens, scale, window, vdim, sinks, gates, mask_chunk, keep_first, softcap, out_scale, out_stride);       \
   } while (0)
   if (dtype == LB_F32) {
     if (vdim <= 256) LB_SIMT(float, 8); else LB_SIMT(float, 20);

@@ -133,6 +133,15 @@ static inline int lb_launch(void (*kernel)(KArgs...), dim3 grid, dim3 block, siz
 // kernel and the fused projection epilogue both take it (the same expression, so the same bits).
 __device__ __forceinline__ float lb_square_pair(float lo, float hi) { return lo * lo + hi * hi; }
 
+// A gated activation whose inputs are clipped: g * sigmoid(slope g) * (u + 1) with g at most `limit` and u within
+// +- limit; 32-bit, rounded by whoever stores it.
+struct LbClip { float limit, slope; };
+__device__ __forceinline__ float lb_clipped_gate(float g, float u, LbClip clip) {
+  g = fminf(g, clip.limit);
+  u = fminf(fmaxf(u, -clip.limit), clip.limit);
+  return g / (1.0f + expf(-clip.slope * g)) * (u + 1.0f);
+}
+
 // Thread-block clusters: blocks that hold parts of one result are launched as one cluster and hand
 // their partial sums to one another through distributed shared memory.
 // LAYOVER_B200_CLUSTER_REDUCE=0 sends split results through scratch memory and a counter instead.

@@ -464,13 +464,14 @@ LB_EXPORT int lb_qk_norm_rope_kv(int dtype, void* qkv, void* q_out, void* k_pool
 // features ([b gates | b ups | b gates | ...]), the layout of the products' fused epilogue.
 // ACT 0: silu (above); ACT 1: relu (max(z, 0), exact in T, so only the product rounds);
 // ACT 2: the tanh form of gelu, 0.5 z (1 + tanh(sqrt(2 / pi) (z + 0.044715 z^3))).
+// ACT 3: the clipped gate (`lb_clipped_gate`), 32-bit to the store.
 template <int ACT> __device__ __forceinline__ float gate_activation(float g) {
   if (ACT == 2) return 0.5f * g * (1.0f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g)));
   return ACT == 1 ? fmaxf(g, 0.f) : g / (1.0f + expf(-g));
 }
 
 template <typename T, bool VEC, int ACT = 0>
-__global__ void swiglu_kernel(const T* __restrict__ gate_up, T* __restrict__ out, long total, int inter, int block) {
+__global__ void swiglu_kernel(const T* __restrict__ gate_up, T* __restrict__ out, long total, int inter, int block, LbClip clip) {
   pdl_launch_dependents();
   pdl_wait();
   constexpr int N = VEC ? Pack<T>::N : 1;
@@ -485,24 +486,25 @@ __global__ void swiglu_kernel(const T* __restrict__ gate_up, T* __restrict__ out
     Pack<T>::load(gp, g);
     Pack<T>::load(gp + up_at, u);
 #pragma unroll
-    for (int i = 0; i < Pack<T>::N; ++i) g[i] = Elem<T>::round(gate_activation<ACT>(g[i])) * u[i];
+    for (int i = 0; i < Pack<T>::N; ++i)
+      g[i] = ACT == 3 ? lb_clipped_gate(g[i], u[i], clip) : Elem<T>::round(gate_activation<ACT>(g[i])) * u[i];
     Pack<T>::store(out + idx, g);
   } else {
     const float g = Elem<T>::load(gp), u = Elem<T>::load(gp + up_at);
-    Elem<T>::store(out + idx, Elem<T>::round(gate_activation<ACT>(g)) * u);
+    Elem<T>::store(out + idx, ACT == 3 ? lb_clipped_gate(g, u, clip) : Elem<T>::round(gate_activation<ACT>(g)) * u);
   }
 }
 
 template <typename T, int ACT = 0>
-static int launch_swiglu(const void* gate_up, void* out, long total, int inter, int block, cudaStream_t stream) {
+static int launch_swiglu(const void* gate_up, void* out, long total, int inter, int block, cudaStream_t stream, LbClip clip = LbClip{}) {
   constexpr int N = Pack<T>::N;
   const bool vec = inter % N == 0 && (block == 0 || block % N == 0) && (uintptr_t)gate_up % 16 == 0 &&
                    (uintptr_t)out % 16 == 0;
   const int threads = 256;
   const long work = vec ? total / N : total;
   const unsigned blocks = (unsigned)((work + threads - 1) / threads);
-  if (vec) lb_launch(swiglu_kernel<T, true, ACT>, blocks, threads, 0, stream, (const T*)gate_up, (T*)out, total, inter, block);
-  else lb_launch(swiglu_kernel<T, false, ACT>, blocks, threads, 0, stream, (const T*)gate_up, (T*)out, total, inter, block);
+  if (vec) lb_launch(swiglu_kernel<T, true, ACT>, blocks, threads, 0, stream, (const T*)gate_up, (T*)out, total, inter, block, clip);
+  else lb_launch(swiglu_kernel<T, false, ACT>, blocks, threads, 0, stream, (const T*)gate_up, (T*)out, total, inter, block, clip);
   return lb_last_error();
 }
 
@@ -516,21 +518,25 @@ LB_EXPORT int lb_swiglu(int dtype, const void* gate_up, void* out, int tokens, i
   return LB_ERR_DTYPE;
 }
 
-// The same gated product with the activation named by the caller: act 0 silu, 1 relu, 2 gelu (tanh form).
+// The same gated product with the activation named by the caller: act 0 silu, 1 relu, 2 gelu (tanh form), 3 the
+// clipped gate with the given limit and slope.
 template <typename T>
-static int launch_gated_act(const void* gate_up, void* out, long total, int inter, int block, int act, cudaStream_t stream) {
+static int launch_gated_act(const void* gate_up, void* out, long total, int inter, int block, int act, LbClip clip,
+                            cudaStream_t stream) {
+  if (act == 3) return launch_swiglu<T, 3>(gate_up, out, total, inter, block, stream, clip);
   if (act == 2) return launch_swiglu<T, 2>(gate_up, out, total, inter, block, stream);
   return act ? launch_swiglu<T, 1>(gate_up, out, total, inter, block, stream)
              : launch_swiglu<T, 0>(gate_up, out, total, inter, block, stream);
 }
 
-LB_EXPORT int lb_gated_act(int dtype, const void* gate_up, void* out, int tokens, int inter, int block, int act,
-                           cudaStream_t stream) {
+LB_EXPORT int lb_gated_act(int dtype, const void* gate_up, void* out, int tokens, int inter, int block, int act, float limit,
+                           float slope, cudaStream_t stream) {
   const long total = (long)tokens * inter;
   if (total <= 0) return 0;
-  if (block < 0 || (block > 0 && inter % block) || act < 0 || act > 2) return LB_ERR_SIZE;
-  if (dtype == LB_F32) return launch_gated_act<float>(gate_up, out, total, inter, block, act, stream);
-  if (dtype == LB_BF16) return launch_gated_act<bf16>(gate_up, out, total, inter, block, act, stream);
+  if (block < 0 || (block > 0 && inter % block) || act < 0 || act > 3) return LB_ERR_SIZE;
+  const LbClip clip{limit, slope};
+  if (dtype == LB_F32) return launch_gated_act<float>(gate_up, out, total, inter, block, act, clip, stream);
+  if (dtype == LB_BF16) return launch_gated_act<bf16>(gate_up, out, total, inter, block, act, clip, stream);
   return LB_ERR_DTYPE;
 }
 
@@ -906,6 +912,7 @@ LB_EXPORT int lb_residual_layernorm(int dtype, float* x, const void* delta_a, co
 //   channels i and i + n_freq of every q and k head (i < n_freq) turn by the token's angle i:
 //       (u, w) -> (u cos - w sin, w cos + u sin), cos/sin from table[t] ([T, 2, n_freq]; null: no rotation)
 //       (flags & 1: neighbouring channels 2i and 2i + 1 turn together instead, by angle i)
+//   every q channel *= 1 + temp_coef ln(floor((p + 1) / temp_every) + 1), p = positions[t] (temp_every 0: no such factor)
 //   values: blend 1 stores v (with its bias) to first_v[t] ([T, kv_heads * vdim] floats) and uses it as it is;
 //           blend 2 uses (1 - lambda) v + lambda first_v[t]; blend 0 uses v
 //           (flags & 2: the row holds no v; a value head is its key head as projected, with the key's bias, before
@@ -922,7 +929,8 @@ __global__ void heads_bias_rope_kv_kernel(const float* __restrict__ proj, long r
                                           const float* __restrict__ lambda, int q_heads, int kv_heads, int dim, int vdim,
                                           int page_tokens, int q_room, int k_room, int v_room,
                                           const float* __restrict__ q_norm_w, const float* __restrict__ k_norm_w,
-                                          float norm_eps, int flags) {
+                                          float norm_eps, int flags, const int* __restrict__ positions, float temp_coef,
+                                          int temp_every) {
   extern __shared__ float head_inv[];     // q_heads + kv_heads: 1 / root mean square of every normed head
   pdl_launch_dependents();
   pdl_wait();
@@ -950,6 +958,7 @@ __global__ void heads_bias_rope_kv_kernel(const float* __restrict__ proj, long r
   const int rotated = cs ? 2 * n_freq : 0;
   const int slot = slot_map[t];
   const size_t page = (size_t)(slot / page_tokens), in_page = (size_t)(slot % page_tokens);
+  const float temperature = temp_every > 0 ? 1.0f + temp_coef * logf((float)((positions[t] + 1) / temp_every + 1)) : 1.f;
   // q and k heads share one loop: head index h over q_heads + kv_heads
   const int qk_items = q_heads * q_room + kv_heads * k_room;
   for (int i = threadIdx.x; i < qk_items; i += blockDim.x) {
@@ -976,7 +985,7 @@ __global__ void heads_bias_rope_kv_kernel(const float* __restrict__ proj, long r
         v = first ? v * cs[f] - w * sn[f] : v * cs[f] + w * sn[f];
       }
     }
-    if (is_q) Elem<T>::store(q_out + (size_t)t * q_heads * q_room + j, v);
+    if (is_q) Elem<T>::store(q_out + (size_t)t * q_heads * q_room + j, temp_every > 0 ? v * temperature : v);
     else Elem<T>::store(k_pool + ((page * kv_heads + h) * page_tokens + in_page) * k_room + c, v);
   }
   const float lam = blend == 2 ? *lambda : 0.f;
@@ -999,8 +1008,9 @@ LB_EXPORT int lb_heads_bias_rope_kv(int dtype, const float* proj, long row_strid
                                     int n_freq, const int* slot_map, float* first_v, int blend, const float* lambda,
                                     int tokens, int q_heads, int kv_heads, int dim, int vdim, int page_tokens, int q_room,
                                     int k_room, int v_room, const float* q_norm_w, const float* k_norm_w, float norm_eps,
-                                    int flags, cudaStream_t stream) {
+                                    int flags, const int* positions, float temp_coef, int temp_every, cudaStream_t stream) {
   if (tokens <= 0) return 0;
+  if (temp_every < 0 || (temp_every > 0 && !positions)) return LB_ERR_SIZE;
   if (q_heads <= 0 || kv_heads <= 0 || dim <= 0 || vdim <= 0 || page_tokens <= 0 || q_room < dim || k_room < dim ||
       v_room < vdim || n_freq < 0 || 2 * n_freq > dim || blend < 0 || blend > 2 || (blend && !first_v) ||
       (blend == 2 && !lambda) || ((flags & 2) && vdim != dim))
@@ -1011,11 +1021,13 @@ LB_EXPORT int lb_heads_bias_rope_kv(int dtype, const float* proj, long row_strid
   if (dtype == LB_F32)
     lb_launch(heads_bias_rope_kv_kernel<float>, tokens, threads, smem, stream, proj, row_stride, (float*)q_out, (float*)k_pool,
               (float*)v_pool, q_bias, k_bias, v_bias, table, n_freq, slot_map, first_v, blend, lambda, q_heads, kv_heads, dim,
-              vdim, page_tokens, q_room, k_room, v_room, q_norm_w, k_norm_w, norm_eps, flags);
+              vdim, page_tokens, q_room, k_room, v_room, q_norm_w, k_norm_w, norm_eps, flags, positions, temp_coef,
+              temp_every);
   else if (dtype == LB_BF16)
     lb_launch(heads_bias_rope_kv_kernel<bf16>, tokens, threads, smem, stream, proj, row_stride, (bf16*)q_out, (bf16*)k_pool,
               (bf16*)v_pool, q_bias, k_bias, v_bias, table, n_freq, slot_map, first_v, blend, lambda, q_heads, kv_heads, dim,
-              vdim, page_tokens, q_room, k_room, v_room, q_norm_w, k_norm_w, norm_eps, flags);
+              vdim, page_tokens, q_room, k_room, v_room, q_norm_w, k_norm_w, norm_eps, flags, positions, temp_coef,
+              temp_every);
   else
     return LB_ERR_DTYPE;
   return lb_last_error();

@@ -469,7 +469,10 @@ __global__ void __launch_bounds__(persistent_threads(EPI), Tile<BN, SWAP, PAIR>:
 gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_b,
                     OutT* __restrict__ C, long ldc, int rows_a, int rows_b, const Schedule sch,
                     float* __restrict__ partials, unsigned* __restrict__ counters, bool vector_ok, const HeadsEpilogue he,
-                    const int* __restrict__ tile_b_rows = nullptr) {
+                    const int* __restrict__ tile_b_rows = nullptr, LbClip clip = LbClip{}) {
+  // GATED epilogues: EPI 1, silu(gate) * up, and EPI 3, the clipped gate with `clip`.
+  constexpr bool GATED = EPI == 1 || EPI == 3;
+  auto gate_up = [clip](float g, float u) { return EPI == 3 ? lb_clipped_gate(g, u, clip) : swiglu_bf16(g, u); };
   // GROUPED products (single blocks, tokens on the 128-row side): `tile_b_rows`, one entry per tile of 128 rows of A
   // and one more, written on the device by an earlier kernel. Entry i: the rows of tile i all belong to one group
   // whose weights start at that row of B (B stacks every group's [rows_b, K] matrix). The last entry is the number
@@ -738,7 +741,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
           }
         }
       }
-      if (EPI == 1 && seg.splits == 1) {
+      if (GATED && seg.splits == 1) {
         // columns come as [64 gate | 64 up] per 128: one thread holds both halves of its token's
         // features and writes 64 activations per 128 columns
         for (int half = 0; half * 128 < valid_cols; ++half) {
@@ -749,7 +752,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
             tmem_ld16(lane_base + half * 128 + 64 + cc, u);
             if (m0 + row < rows_a) {
 #pragma unroll
-              for (int i = 0; i < 16; ++i) g[i] = swiglu_bf16(g[i], u[i]);
+              for (int i = 0; i < 16; ++i) g[i] = gate_up(g[i], u[i]);
               OutT* dst = C + (size_t)(m0 + row) * ldc + (n0 >> 1) + half * 64 + cc;
               if (vector_ok) {
                 store_row16<OutT>(dst, g);
@@ -761,7 +764,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
           }
         }
       }
-      for (int c = 0; c < BN && !(EPI == 1 && seg.splits == 1) && EPI != 2; c += 16) {
+      for (int c = 0; c < BN && !(GATED && seg.splits == 1) && EPI != 2; c += 16) {
         if (c >= valid_cols) break;                           // uniform over the block
         float v[16];
         tmem_ld16(lane_base + c, v);
@@ -824,7 +827,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
           const int quads = (valid_cols + 3) >> 2;                      // groups of four columns
           const int share = (quads + seg.splits - 1) / seg.splits;
           const int q_begin = seg.split * share, q_end = min(quads, q_begin + share);
-          if (EPI == 1) {
+          if (GATED) {
             // shares of OUTPUT quads: output quad o of a 128-column half h sums gate quad
             // 32 h + o and up quad 32 h + 16 + o over the splits, then combines them
             const int out_quads = valid_cols >> 3;
@@ -842,10 +845,10 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
                   u.x += pu.x; u.y += pu.y; u.z += pu.z; u.w += pu.w;
                 }
                 OutT* dst = C + (size_t)(m0 + row) * ldc + (n0 >> 1) + oq * 4;
-                store_one<OutT>(dst, swiglu_bf16(g.x, u.x));
-                store_one<OutT>(dst + 1, swiglu_bf16(g.y, u.y));
-                store_one<OutT>(dst + 2, swiglu_bf16(g.z, u.z));
-                store_one<OutT>(dst + 3, swiglu_bf16(g.w, u.w));
+                store_one<OutT>(dst, gate_up(g.x, u.x));
+                store_one<OutT>(dst + 1, gate_up(g.y, u.y));
+                store_one<OutT>(dst + 2, gate_up(g.z, u.z));
+                store_one<OutT>(dst + 3, gate_up(g.w, u.w));
               }
             }
           } else if (m0 + row < rows_a) {
@@ -942,7 +945,7 @@ struct Problem {
 
 template <int BN, bool SWAP, typename OutT, int EPI = 0>
 int launch(const CUtensorMap& map_a, const CUtensorMap& map_b, void* C, long ldc, const Problem& pb, bool vector_ok,
-           cudaStream_t stream, const int* tile_b_rows = nullptr) {
+           cudaStream_t stream, const int* tile_b_rows = nullptr, LbClip clip = LbClip{}) {
   using T = Tile<BN, SWAP>;
   auto kernel = gemm_tcgen05_kernel<BN, SWAP, OutT, EPI>;
   static int blocks_per_sm = 0;      // how many blocks of this kernel an SM really holds (the same on every B200)
@@ -997,7 +1000,7 @@ int launch(const CUtensorMap& map_a, const CUtensorMap& map_b, void* C, long ldc
   float* partials = sch.last_splits > 1 ? pb.scratch : nullptr;
   const int code = lb_launch(kernel, dim3(blocks), dim3(PERSISTENT_THREADS), (size_t)T::SMEM, stream, map_a, map_b,
                              (OutT*)C, ldc, pb.rows_a, pb.rows_b, sch, partials, pb.counters, vector_ok, HeadsEpilogue{},
-                             tile_b_rows);
+                             tile_b_rows, clip);
   return code ? code : lb_last_error();
 }
 
@@ -1073,7 +1076,7 @@ int launch_pair(const CUtensorMap& map_a, const CUtensorMap& map_b, void* C, lon
   float* partials = sch.last_splits > 1 ? pb.scratch : nullptr;
   const int code = lb_launch_cluster_dims(kernel, dim3(2 * pairs), dim3(persistent_threads(EPI)), (size_t)T::SMEM, stream,
                                           dim3(2, 1, 1), map_a, map_b, (OutT*)C, ldc, pb.rows_a, pb.rows_b, sch, partials,
-                                          pb.counters, vector_ok, he, (const int*)nullptr);
+                                          pb.counters, vector_ok, he, (const int*)nullptr, LbClip{});
   return code ? code : lb_last_error();
 }
 
@@ -1273,15 +1276,16 @@ LB_EXPORT int lb_gemm_tcgen05(const void* A, const void* W, void* C, int out_dty
 // stream) holds g * N for a tile of group g; its last entry is the number of row tiles in use (all at the front,
 // the tiles behind them cost nothing). M is the
 // number of rows A and C have room for (a multiple of 128 that the host knows without asking the device).
-// Always the many-token orientation on single blocks; `epilogue` as in `lb_gemm_tcgen05`.
+// Always the many-token orientation on single blocks; `epilogue` as in `lb_gemm_tcgen05`, and 3: the same row blocks
+// with the clipped gate of `limit` and `slope`.
 LB_EXPORT int lb_gemm_tcgen05_grouped(const void* A, const void* W, void* C, int out_dtype, int M, int N, int K, int groups,
                                       long lda, long ldw, long ldc, const int* tile_b_rows, float* scratch,
                                       long scratch_floats, unsigned* counters, int n_counters, int sm_count, int epilogue,
-                                      cudaStream_t stream) {
+                                      float limit, float slope, cudaStream_t stream) {
   if (M <= 0 || N <= 0) return 0;
   if (M % BM || groups <= 0 || !tile_b_rows) return LB_ERR_SIZE;
-  if (epilogue != 0 && epilogue != 1) return LB_ERR_SIZE;
-  if (epilogue == 1 && (N % 128 != 0 || out_dtype != LB_BF16)) return LB_ERR_SIZE;
+  if (epilogue != 0 && epilogue != 1 && epilogue != 3) return LB_ERR_SIZE;
+  if (epilogue && (N % 128 != 0 || out_dtype != LB_BF16)) return LB_ERR_SIZE;
   if (!lb_gemm_tcgen05_supports(A, W, K, lda, ldw)) return LB_ERR_ALIGN;
   if (out_dtype != LB_BF16 && out_dtype != LB_F32) return LB_ERR_DTYPE;
   if (sm_count < 1) sm_count = 1;
@@ -1294,6 +1298,11 @@ LB_EXPORT int lb_gemm_tcgen05_grouped(const void* A, const void* W, void* C, int
   if (epilogue == 1) {
     if (bn == 128) return launch<128, false, bf16, 1>(map_a, map_b, C, ldc, pb, vector_ok, stream, tile_b_rows);
     return launch<256, false, bf16, 1>(map_a, map_b, C, ldc, pb, vector_ok, stream, tile_b_rows);
+  }
+  if (epilogue == 3) {
+    const LbClip clip{limit, slope};
+    if (bn == 128) return launch<128, false, bf16, 3>(map_a, map_b, C, ldc, pb, vector_ok, stream, tile_b_rows, clip);
+    return launch<256, false, bf16, 3>(map_a, map_b, C, ldc, pb, vector_ok, stream, tile_b_rows, clip);
   }
   if (out_dtype == LB_BF16) {
     if (bn == 128) return launch<128, false, bf16>(map_a, map_b, C, ldc, pb, vector_ok, stream, tile_b_rows);

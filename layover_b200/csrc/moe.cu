@@ -5,12 +5,14 @@
 //
 //   route     z = W_router h in 32-bit, one warp per token; score = sigmoid(z); the `top` largest z
 //             (ties: the lower index) with their scores; optionally one more 32-bit dot product per
-//             token, sigmoid(w_shared . h), the factor of a shared expert
+//             token, sigmoid(w_shared . h), the factor of a shared expert; or the scores are the softmax over
+//             the chosen logits alone
 //   group     offsets[e] .. offsets[e + 1] = the places of expert e's pairs in `order`, order[place] =
 //             pair = token * top + k
 //   products  for every expert e and every pair in its group
 //               up    act[place]  = T(act_fn(s * (Wg_e h)) * (s * (Wu_e h)))   s = the pair's score
 //               down  y[pair]     = Wd_e act[place]                             (32-bit)
+//             or, with clipped gates, act[place] = T(lb_clipped_gate(s Wg_e h, s Wu_e h))
 //             The score multiplies the expert's INPUT; W (s h) = s (W h), and the factor is applied to
 //             the 32-bit sums rather than to a rounded s h. Every output element is one dot product
 //             summed in the order of k, so it does not depend on where its row sits in a tile or on
@@ -63,11 +65,14 @@ template <> struct Piece<bf16> {
 //               chosen (ties: the lower index)
 //   renorm      the chosen weights are divided by their sum (+ 1e-20)
 //   scale       then multiplied by this
+//   softmax     the choice is made on the logits and the weights are the softmax over the chosen logits; with none of
+//               the others
 // All of it is one warp's work per token on 32-bit numbers in shared memory.
 struct RouteOptions {
   const float* correction;
   int groups, keep, renorm;
   float scale;
+  int softmax;
   __host__ __device__ bool general() const { return correction || groups > 1 || renorm || scale != 1.f; }
 };
 
@@ -139,6 +144,19 @@ __device__ __forceinline__ void choose_general(float* z, float* s, float* g, int
     const float factor = (opt.renorm ? 1.0f / (sum + 1e-20f) : 1.f) * opt.scale;
     for (int k = 0; k < top; ++k) scores[k] *= factor;
   }
+}
+
+// The chosen logits (largest first) become their softmax. One thread.
+__device__ __forceinline__ void softmax_chosen(float* scores, int top) {
+  const float largest = scores[0];
+  float sum = 0.f;
+  for (int k = 0; k < top; ++k) {
+    const float e = expf(scores[k] - largest);
+    scores[k] = e;
+    sum += e;
+  }
+  const float inv = 1.0f / sum;
+  for (int k = 0; k < top; ++k) scores[k] *= inv;
 }
 
 // A block takes TT tokens; its warps share the experts (warp w takes experts w, w + WARPS, ...) and one more row for the
@@ -224,11 +242,12 @@ moe_route_kernel(const T* __restrict__ h, const float* __restrict__ router, cons
       if (at >= experts) at = k;                    // only when every logit left is NaN or -inf
       if (lane == 0) {
         ids[(size_t)(t0 + t) * top + k] = at;
-        scores[(size_t)(t0 + t) * top + k] = 1.0f / (1.0f + expf(-best));
+        scores[(size_t)(t0 + t) * top + k] = opt.softmax ? best : 1.0f / (1.0f + expf(-best));
         z[at] = -INFINITY;                          // taken
       }
       __syncwarp();
     }
+    if (opt.softmax && lane == 0) softmax_chosen(scores + (size_t)(t0 + t) * top, top);
   }
 }
 
@@ -271,11 +290,12 @@ moe_select_kernel(const float* __restrict__ logits, long stride, int* __restrict
     if (at >= experts) at = k;                      // only when every logit left is NaN or -inf
     if (lane == 0) {
       ids[(size_t)t * top + k] = at;
-      scores[(size_t)t * top + k] = 1.0f / (1.0f + expf(-best));
+      scores[(size_t)t * top + k] = opt.softmax ? best : 1.0f / (1.0f + expf(-best));
       z[at] = -INFINITY;                            // taken
     }
     __syncwarp();
   }
+  if (opt.softmax && lane == 0) softmax_chosen(scores + (size_t)t * top, top);
 }
 
 // One block: count, scan, place. The order inside a group is the order of arrival; no result depends on it.
@@ -378,6 +398,11 @@ template <int ACT> __device__ __forceinline__ float expert_activation(float g) {
   return g / (1.0f + expf(-g));      // silu
 }
 
+// ACT 0 silu, 1 relu, 2 relu squared: act(g) * u. ACT 3: the clipped gate.
+template <int ACT> __device__ __forceinline__ float expert_gate(float g, float u, LbClip clip) {
+  return ACT == 3 ? lb_clipped_gate(g, u, clip) : expert_activation<ACT>(g) * u;
+}
+
 // The experts' products on the FFMA pipes (both precisions; 32-bit sums). A block owns BM places of one
 // expert's group and BN output columns; a thread TM x TN of them. The k loop runs in steps of BK through
 // shared memory, every element's sum in the order of k.
@@ -391,7 +416,7 @@ moe_expert_product_kernel(const T* __restrict__ a, long a_stride, const int* __r
                           const int* __restrict__ offsets, int experts, const T* __restrict__ w, long expert_stride,
                           int n_out, int k_dim, OutT* __restrict__ out, long out_stride,
                           const int* __restrict__ out_rows, const float* __restrict__ pair_scale,
-                          const int* __restrict__ order, int interleaved) {
+                          const int* __restrict__ order, int interleaved, LbClip clip) {
   constexpr int BK = 32, THREADS = (BM / TM) * (BN / TN);
   __shared__ float a_s[BK][BM + 1];
   __shared__ float w_s[GATED ? 2 : 1][BK][BN + 1];
@@ -467,7 +492,7 @@ moe_expert_product_kernel(const T* __restrict__ a, long a_stride, const int* __r
     for (int j = 0; j < TN; ++j) {
       const int n = n0 + tx + j * (BN / TN);
       if (n >= n_out) continue;
-      if (GATED) Elem<OutT>::store(out + dst * out_stride + n, expert_activation<ACT>(s * acc[0][i][j]) * (s * acc[GATED ? 1 : 0][i][j]));
+      if (GATED) Elem<OutT>::store(out + dst * out_stride + n, expert_gate<ACT>(s * acc[0][i][j], s * acc[GATED ? 1 : 0][i][j], clip));
       else Elem<OutT>::store(out + dst * out_stride + n, ACT == 2 ? expert_activation<2>(acc[0][i][j]) : acc[0][i][j]);
     }
   }
@@ -486,7 +511,7 @@ moe_expert_rows_kernel(const T* __restrict__ a, long a_stride, const int* __rest
                        const int* __restrict__ offsets, int experts, const T* __restrict__ w, long expert_stride,
                        int n_out, int k_dim, OutT* __restrict__ out, long out_stride,
                        const int* __restrict__ out_rows, const float* __restrict__ pair_scale,
-                       const int* __restrict__ order, int interleaved, int features_per_warp) {
+                       const int* __restrict__ order, int interleaved, LbClip clip, int features_per_warp) {
   constexpr int N = Piece<T>::N, Z = GATED ? 2 : 1, F = FEW_FEATURES;
   __shared__ int found[3];
   __shared__ long row_of[FEW_ROWS];
@@ -564,7 +589,7 @@ moe_expert_rows_kernel(const T* __restrict__ a, long a_stride, const int* __rest
             const long dst = out_rows ? out_rows[place] : place;
             if (GATED) {
               const float sc = pair_scale ? pair_scale[order[place]] : 1.f;
-              Elem<OutT>::store(out + dst * out_stride + n0 + f, expert_activation<ACT>(sc * g) * (sc * u));
+              Elem<OutT>::store(out + dst * out_stride + n0 + f, expert_gate<ACT>(sc * g, sc * u, clip));
             } else {
               Elem<OutT>::store(out + dst * out_stride + n0 + f, ACT == 2 ? expert_activation<2>(g) : g);
             }
@@ -598,9 +623,9 @@ template <typename T, bool GATED, typename OutT>
 int launch_product(bool few, int act, const void* a, long a_stride, const int* a_rows, int a_div, const int* offsets,
                    int experts, const void* w, long expert_stride, int n_out, int k_dim, void* out, long out_stride,
                    const int* out_rows, const float* pair_scale, const int* order, int n_pairs, cudaStream_t stream,
-                   int interleaved = 0) {
+                   int interleaved = 0, LbClip clip = LbClip{}) {
 #define LB_MOE_ARGS (const T*)a, a_stride, a_rows, a_div, offsets, experts, (const T*)w, expert_stride, n_out, k_dim, \
-                    (OutT*)out, out_stride, out_rows, pair_scale, order, interleaved
+                    (OutT*)out, out_stride, out_rows, pair_scale, order, interleaved, clip
   const bool aligned = (uintptr_t)a % 16 == 0 && (uintptr_t)w % 16 == 0 && k_dim % Piece<T>::N == 0 &&
                        (a_stride * sizeof(T)) % 16 == 0;
   if (few && aligned) {     // a handful of rows per expert: a stream of the chosen experts' weight rows
@@ -610,21 +635,24 @@ int launch_product(bool few, int act, const void* a, long a_stride, const int* a
     int per_warp = 8;
     while (per_warp > FEW_FEATURES && (long)tiles * ((n_out + FEW_WARPS * per_warp - 1) / (FEW_WARPS * per_warp)) < 4 * 148) per_warp >>= 1;
     dim3 grid(tiles, (n_out + FEW_WARPS * per_warp - 1) / (FEW_WARPS * per_warp));
-    if (act == 1) lb_launch(moe_expert_rows_kernel<T, OutT, GATED, 1>, grid, FEW_WARPS * 32, (size_t)experts * sizeof(int), stream, LB_MOE_ARGS, per_warp);
+    if (GATED && act == 3) lb_launch(moe_expert_rows_kernel<T, OutT, GATED, GATED ? 3 : 0>, grid, FEW_WARPS * 32, (size_t)experts * sizeof(int), stream, LB_MOE_ARGS, per_warp);
+    else if (act == 1) lb_launch(moe_expert_rows_kernel<T, OutT, GATED, 1>, grid, FEW_WARPS * 32, (size_t)experts * sizeof(int), stream, LB_MOE_ARGS, per_warp);
     else if (act == 2) lb_launch(moe_expert_rows_kernel<T, OutT, GATED, 2>, grid, FEW_WARPS * 32, (size_t)experts * sizeof(int), stream, LB_MOE_ARGS, per_warp);
     else lb_launch(moe_expert_rows_kernel<T, OutT, GATED, 0>, grid, FEW_WARPS * 32, (size_t)experts * sizeof(int), stream, LB_MOE_ARGS, per_warp);
   } else if (few) {      // the same through tiles of 8 places, for sizes and addresses that cannot be read 16 bytes at a time
     constexpr int BM = 8, BN = 128;
     dim3 grid((n_pairs + BM - 1) / BM + experts, (n_out + BN - 1) / BN);
     if (grid.x > (unsigned)n_pairs) grid.x = n_pairs;   // every tile holds a pair
-    if (act == 1) lb_launch(moe_expert_product_kernel<T, OutT, BM, BN, 1, 4, GATED, 1>, grid, 256, (size_t)experts * sizeof(int), stream, LB_MOE_ARGS);
+    if (GATED && act == 3) lb_launch(moe_expert_product_kernel<T, OutT, BM, BN, 1, 4, GATED, GATED ? 3 : 0>, grid, 256, (size_t)experts * sizeof(int), stream, LB_MOE_ARGS);
+    else if (act == 1) lb_launch(moe_expert_product_kernel<T, OutT, BM, BN, 1, 4, GATED, 1>, grid, 256, (size_t)experts * sizeof(int), stream, LB_MOE_ARGS);
     else if (act == 2) lb_launch(moe_expert_product_kernel<T, OutT, BM, BN, 1, 4, GATED, 2>, grid, 256, (size_t)experts * sizeof(int), stream, LB_MOE_ARGS);
     else lb_launch(moe_expert_product_kernel<T, OutT, BM, BN, 1, 4, GATED, 0>, grid, 256, (size_t)experts * sizeof(int), stream, LB_MOE_ARGS);
   } else {
     constexpr int BM = 64, BN = 64;
     dim3 grid((n_pairs + BM - 1) / BM + experts, (n_out + BN - 1) / BN);
     if (grid.x > (unsigned)n_pairs) grid.x = n_pairs;
-    if (act == 1) lb_launch(moe_expert_product_kernel<T, OutT, BM, BN, 4, 4, GATED, 1>, grid, 256, (size_t)experts * sizeof(int), stream, LB_MOE_ARGS);
+    if (GATED && act == 3) lb_launch(moe_expert_product_kernel<T, OutT, BM, BN, 4, 4, GATED, GATED ? 3 : 0>, grid, 256, (size_t)experts * sizeof(int), stream, LB_MOE_ARGS);
+    else if (act == 1) lb_launch(moe_expert_product_kernel<T, OutT, BM, BN, 4, 4, GATED, 1>, grid, 256, (size_t)experts * sizeof(int), stream, LB_MOE_ARGS);
     else if (act == 2) lb_launch(moe_expert_product_kernel<T, OutT, BM, BN, 4, 4, GATED, 2>, grid, 256, (size_t)experts * sizeof(int), stream, LB_MOE_ARGS);
     else lb_launch(moe_expert_product_kernel<T, OutT, BM, BN, 4, 4, GATED, 0>, grid, 256, (size_t)experts * sizeof(int), stream, LB_MOE_ARGS);
   }
@@ -657,19 +685,21 @@ static void launch_route(const void* h, const float* router, const float* shared
 #undef LB_ROUTE_ARGS
 }
 
-static bool route_options(RouteOptions& opt, const float* correction, int groups, int keep, int renorm, float scale, int experts) {
-  opt = RouteOptions{correction, groups > 1 ? groups : 0, keep, renorm, scale};
+static bool route_options(RouteOptions& opt, const float* correction, int groups, int keep, int renorm, float scale, int softmax,
+                          int experts) {
+  opt = RouteOptions{correction, groups > 1 ? groups : 0, keep, renorm, scale, softmax};
+  if (softmax && opt.general()) return false;
   return !(groups > 1 && (experts % groups || keep <= 0 || keep > groups)) && scale > 0.f;
 }
 
-// correction, groups, keep, renorm, scale: see RouteOptions (null, 0, 0, 0, 1: the `top` largest logits and their sigmoids).
+// correction, groups, keep, renorm, scale, softmax: see RouteOptions (null, 0, 0, 0, 1, 0: the `top` largest logits and their sigmoids).
 LB_EXPORT int lb_moe_route(int dtype, const void* h, const float* router, const float* shared_w, int* ids, float* scores,
                            float* shared_factor, int tokens, int hidden, int experts, int top, const float* correction,
-                           int groups, int keep, int renorm, float scale, cudaStream_t stream) {
+                           int groups, int keep, int renorm, float scale, int softmax, cudaStream_t stream) {
   if (tokens <= 0) return 0;
   RouteOptions opt;
   if (hidden <= 0 || experts <= 0 || top <= 0 || top > experts || experts > 1024 || (shared_w && !shared_factor) ||
-      !route_options(opt, correction, groups, keep, renorm, scale, experts))
+      !route_options(opt, correction, groups, keep, renorm, scale, softmax, experts))
     return LB_ERR_SIZE;
   if (dtype == LB_F32) launch_route<float>(h, router, shared_w, ids, scores, shared_factor, tokens, hidden, experts, top, opt, stream);
   else if (dtype == LB_BF16) launch_route<bf16>(h, router, shared_w, ids, scores, shared_factor, tokens, hidden, experts, top, opt, stream);
@@ -681,11 +711,11 @@ LB_EXPORT int lb_moe_route(int dtype, const void* h, const float* router, const 
 // stride `stride` floats.
 LB_EXPORT int lb_moe_select(const float* logits, long stride, int* ids, float* scores, float* shared_factor, int tokens,
                             int experts, int top, const float* correction, int groups, int keep, int renorm, float scale,
-                            cudaStream_t stream) {
+                            int softmax, cudaStream_t stream) {
   if (tokens <= 0) return 0;
   RouteOptions opt;
   if (experts <= 0 || top <= 0 || top > experts || experts > 1024 || stride < experts + (shared_factor ? 1 : 0) ||
-      !route_options(opt, correction, groups, keep, renorm, scale, experts))
+      !route_options(opt, correction, groups, keep, renorm, scale, softmax, experts))
     return LB_ERR_SIZE;
   lb_launch(moe_select_kernel, (tokens + SELECT_WARPS - 1) / SELECT_WARPS, SELECT_WARPS * 32,
             (size_t)SELECT_WARPS * (experts + (opt.general() ? experts + opt.groups : 0)) * sizeof(float), stream, logits, stride, ids,
@@ -702,13 +732,15 @@ LB_EXPORT int lb_moe_group(const int* ids, int n_pairs, int experts, int* offset
 
 // act[place, :] = T(act_fn(s g) * (s u)) for every place of `order`: h [tokens, hidden] (row stride h_stride), gate_up
 // [experts, 2 * inter, hidden] (gate rows, then up rows; `interleaved`: blocks of 64 gate rows + the 64 up rows of the same
-// features), scores by pair (null: s = 1). activation 0 silu, 1 relu, 2 the square of relu. gated 0: the experts have no
+// features), scores by pair (null: s = 1). activation 0 silu, 1 relu, 2 the square of relu, 3 the clipped gate
+// (act[place, :] = T(lb_clipped_gate(s g, s u)) with `limit` and `slope`). gated 0: the experts have no
 // gate; gate_up is [experts, inter, hidden] and act[place, :] = T(relu(up_e h)^2) (activation 2 only, no scores).
 LB_EXPORT int lb_moe_expert_up(int dtype, const void* h, long h_stride, const int* order, const int* offsets,
                                const float* scores, const void* gate_up, void* act, int n_pairs, int top, int experts,
-                               int hidden, int inter, int activation, int interleaved, int gated, cudaStream_t stream) {
+                               int hidden, int inter, int activation, int interleaved, int gated, float limit, float slope,
+                               cudaStream_t stream) {
   if (n_pairs <= 0) return 0;
-  if (experts <= 0 || experts > 1024 || hidden <= 0 || inter <= 0 || top <= 0 || activation < 0 || activation > 2) return LB_ERR_SIZE;
+  if (experts <= 0 || experts > 1024 || hidden <= 0 || inter <= 0 || top <= 0 || activation < 0 || activation > 3) return LB_ERR_SIZE;
   if (interleaved && inter % 64) return LB_ERR_SIZE;
   const bool few = n_pairs <= 4 * experts;
   if (!gated) {
@@ -724,10 +756,10 @@ LB_EXPORT int lb_moe_expert_up(int dtype, const void* h, long h_stride, const in
   const long expert_stride = 2L * inter * hidden;
   if (dtype == LB_F32)
     return launch_product<float, true, float>(few, activation, h, h_stride, order, top, offsets, experts, gate_up, expert_stride,
-                                              inter, hidden, act, inter, nullptr, scores, order, n_pairs, stream, interleaved);
+                                              inter, hidden, act, inter, nullptr, scores, order, n_pairs, stream, interleaved, LbClip{limit, slope});
   if (dtype == LB_BF16)
     return launch_product<bf16, true, bf16>(few, activation, h, h_stride, order, top, offsets, experts, gate_up, expert_stride,
-                                            inter, hidden, act, inter, nullptr, scores, order, n_pairs, stream, interleaved);
+                                            inter, hidden, act, inter, nullptr, scores, order, n_pairs, stream, interleaved, LbClip{limit, slope});
   return LB_ERR_DTYPE;
 }
 

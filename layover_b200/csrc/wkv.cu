@@ -1,5 +1,6 @@
-// Time mixing with a decay per key channel that depends on the token (the WKV recurrence), as kernels over
-// the requests' state rows.
+// Recurrences with a decay per key channel that depends on the token, as kernels over the requests' state rows: time
+// mixing (the WKV recurrence, which reads its state before the token's own write and adds a bonus for it) and gated
+// linear attention (which reads after the write).
 //
 // A request's state row (32-bit floats): S of every head [heads, dim, dim] (key channel, value channel), then
 // the previous token's input h [width].
@@ -11,12 +12,16 @@
 //   scan          per head:  o_t = (S + diag(u) k_t v_t^T)^T r_t,   S <- diag(w_t) S + k_t v_t^T
 //                 o_t[e] = sum_d r_t[d] (S[d, e] + u[d] k_t[d] v_t[e])
 //
+// Gated linear attention has no shift; its state row is S [heads, dim, vdim] alone, and
+//   decay         w[t, c] = sigmoid(w0[c] + sum_j W2[c, j] a[t, j])^(1 / tau)
+//   scan          per head:  S <- diag(w_t) S + k_t v_t^T,   o_t = scale * S^T q_t          (values of their own size)
+//
 // One scan kernel serves a whole prompt, a portion of one and a single decoded token: a sequence's tokens of the
 // step are walked in order from the state the step before left. Every state element takes the same operations
 // whatever the cut, and the sums over d run in an order that depends on the head size alone, so results do not
 // depend on how the tokens were cut into steps or on what else is in the batch, bit for bit.
 //
-// Scan grid (ceil(dim / 16), heads, sequences), 8 warps (heads of up to 32 channels: 32 columns a block): a block owns
+// Scan grid (ceil(vdim / 16), heads, sequences), 8 warps (heads of up to 32 channels: 32 columns a block): a block owns
 // 16 columns of one head's S, a thread DPT rows of one column (16 groups of rows a block, two a warp), so a lone
 // prompt of 16 heads of 128 is 128 blocks. Tokens come CHUNK at a time through two shared-memory buffers filled by
 // cp.async while the chunk before is worked on; r, k, w are read as 16-byte broadcasts; each group of rows leaves its
@@ -102,11 +107,12 @@ __global__ void wkv_shift_tail_kernel(const T* __restrict__ h, float* __restrict
 }
 
 // DECAY_TOKENS tokens a block share every weight they read; a thread owns channels, its sum runs in the order of j. The
-// tokens' tanh(a) sit in shared memory, rows padded with zeros to whole 16-byte pieces that every thread reads at once.
-template <typename T, bool VEC>
+// tokens' tanh(a) (GATE: a itself) sit in shared memory, rows padded with zeros to whole 16-byte pieces that every thread reads at once.
+// GATE: the finish is sigmoid(z)^(1 / tau) = exp(-softplus(-z) / tau) instead of exp(-exp(z)).
+template <typename T, bool VEC, bool GATE>
 __global__ void __launch_bounds__(256)
 wkv_decay_kernel(const float* __restrict__ a, long a_stride, const T* __restrict__ w2, const float* __restrict__ w0,
-                 float* __restrict__ decay, int tokens, int channels, int rank) {
+                 float* __restrict__ decay, int tokens, int channels, int rank, float inv_tau) {
   extern __shared__ __align__(16) float z_s[];     // [DECAY_TOKENS][padded rank]
   pdl_launch_dependents();
   pdl_wait();
@@ -114,7 +120,9 @@ wkv_decay_kernel(const float* __restrict__ a, long a_stride, const T* __restrict
   const int t0 = blockIdx.x * DECAY_TOKENS, n = min(DECAY_TOKENS, tokens - t0);
   for (int i = threadIdx.x; i < DECAY_TOKENS * padded; i += blockDim.x) {
     const int t = i / padded, j = i - t * padded;
-    z_s[i] = (t < n && j < rank) ? tanhf(a[(size_t)(t0 + t) * a_stride + j]) : 0.f;
+    float z = 0.f;
+    if (t < n && j < rank) z = a[(size_t)(t0 + t) * a_stride + j];
+    z_s[i] = GATE ? z : tanhf(z);
   }
   __syncthreads();
   for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < channels; c += gridDim.y * blockDim.x) {
@@ -144,7 +152,11 @@ wkv_decay_kernel(const float* __restrict__ a, long a_stride, const T* __restrict
     const float bias = w0[c];
 #pragma unroll
     for (int t = 0; t < DECAY_TOKENS; ++t)
-      if (t < n) decay[(size_t)(t0 + t) * channels + c] = expf(-expf(acc[t] + bias));
+      if (t < n) {
+        const float z = acc[t] + bias;
+        const float minus_log = GATE ? (fmaxf(-z, 0.f) + log1pf(expf(-fabsf(z)))) * inv_tau : expf(z);
+        decay[(size_t)(t0 + t) * channels + c] = expf(-minus_log);
+      }
   }
 }
 
@@ -157,16 +169,17 @@ __device__ __forceinline__ void copy_async_16(float* dst_shared, const float* sr
 __device__ __forceinline__ void copy_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
 template <int N> __device__ __forceinline__ void copy_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
 
-// r, k, v float [T, *] with row strides; w float [T, heads * dim]; u float [heads, dim]; out float [T, heads * dim].
+// r, k, v float [T, *] with row strides; w float [T, heads * dim]; u float [heads, dim]; out float [T, heads * vdim].
+// AFTER: the state is read after the token's own write, without a bonus (u unused), and the sum is multiplied by `scale`.
 // COLS value columns a block (16, or 32 for small heads); a warp holds 32 / COLS groups of rows of them, a block
 // GROUPS = 8 * 32 / COLS groups of DPT rows each. VEC: dim is a multiple of 4 and every row of r, k, w starts on a
 // 16-byte boundary.
-template <int DPT, int COLS, bool VEC>
+template <int DPT, int COLS, bool VEC, bool AFTER>
 __global__ void __launch_bounds__(SCAN_THREADS, DPT <= 8 ? 3 : 1)      // single tokens are bound by the state's traffic: three blocks an SM keep it in flight
 wkv_scan_kernel(const float* __restrict__ r, long r_stride, const float* __restrict__ k, long k_stride,
                 const float* __restrict__ v, long v_stride, const float* __restrict__ w, const float* __restrict__ u,
                 float* __restrict__ out, float* __restrict__ state, long state_stride, const int* __restrict__ cu_q,
-                const int* __restrict__ state_slots, int heads, int dim) {
+                const int* __restrict__ state_slots, int heads, int dim, int vdim, float scale) {
   static_assert(DPT % 4 == 0, "16-byte broadcasts");
   constexpr int GROUPS = RANGES * (32 / COLS), DPAD = GROUPS * DPT;
   extern __shared__ __align__(16) float wkv_smem[];
@@ -182,15 +195,15 @@ wkv_scan_kernel(const float* __restrict__ r, long r_stride, const float* __restr
   pdl_wait();
   const int first = cu_q[seq], count = cu_q[seq + 1] - first;
   if (count <= 0) return;
-  float* mine = state + (size_t)state_slots[seq] * state_stride + (size_t)head * dim * dim;
+  float* mine = state + (size_t)state_slots[seq] * state_stride + (size_t)head * dim * vdim;
   float s[DPT], bonus[DPT];
 #pragma unroll
   for (int x = 0; x < DPT; ++x) {
     const int d = d0 + x;
-    s[x] = (d < dim && e < dim) ? mine[(size_t)d * dim + e] : 0.f;
-    bonus[x] = d < dim ? u[(size_t)head * dim + d] : 0.f;
+    s[x] = (d < dim && e < vdim) ? mine[(size_t)d * vdim + e] : 0.f;
+    bonus[x] = (!AFTER && d < dim) ? u[(size_t)head * dim + d] : 0.f;
   }
-  const size_t col0 = (size_t)head * dim;
+  const size_t col0 = (size_t)head * dim, vcol0 = (size_t)head * vdim;
   // which 16-byte pieces of a chunk's r, k and w rows this thread copies: the same for every chunk, worked out once
   constexpr int PIECES_EACH = (CHUNK * DPAD / 4 + SCAN_THREADS - 1) / SCAN_THREADS;
   int piece_t[PIECES_EACH], piece_d[PIECES_EACH];
@@ -222,7 +235,7 @@ wkv_scan_kernel(const float* __restrict__ r, long r_stride, const float* __restr
     }
     for (int i = threadIdx.x; i < n * COLS; i += SCAN_THREADS) {
       const int t = i / COLS, c = i - t * COLS;
-      if (e0 + c < dim) copy_async_4(&v_s[buf][t][c], v + (size_t)(first + t0 + t) * v_stride + col0 + e0 + c);
+      if (e0 + c < vdim) copy_async_4(&v_s[buf][t][c], v + (size_t)(first + t0 + t) * v_stride + vcol0 + e0 + c);
     }
     copy_async_commit();
   };
@@ -245,6 +258,13 @@ wkv_scan_kernel(const float* __restrict__ r, long r_stride, const float* __restr
         const float4 rr = *reinterpret_cast<const float4*>(&rkw_s[buf][0][t][d0 + x]);
         const float4 kk = *reinterpret_cast<const float4*>(&rkw_s[buf][1][t][d0 + x]);
         const float4 ww = *reinterpret_cast<const float4*>(&rkw_s[buf][2][t][d0 + x]);
+        if (AFTER) {
+          s[x] = fmaf(ww.x, s[x], kk.x * vt); p0 = fmaf(rr.x, s[x], p0);
+          s[x + 1] = fmaf(ww.y, s[x + 1], kk.y * vt); p1 = fmaf(rr.y, s[x + 1], p1);
+          s[x + 2] = fmaf(ww.z, s[x + 2], kk.z * vt); p0 = fmaf(rr.z, s[x + 2], p0);
+          s[x + 3] = fmaf(ww.w, s[x + 3], kk.w * vt); p1 = fmaf(rr.w, s[x + 3], p1);
+          continue;
+        }
         float kv;
         kv = kk.x * vt; p0 = fmaf(rr.x, fmaf(bonus[x], kv, s[x]), p0); s[x] = fmaf(ww.x, s[x], kv);
         kv = kk.y * vt; p1 = fmaf(rr.y, fmaf(bonus[x + 1], kv, s[x + 1]), p1); s[x + 1] = fmaf(ww.y, s[x + 1], kv);
@@ -262,39 +282,39 @@ wkv_scan_kernel(const float* __restrict__ r, long r_stride, const float* __restr
     __syncthreads();
     if (threadIdx.x < n * COLS) {
       const int t = threadIdx.x / COLS, c = threadIdx.x - t * COLS;
-      if (e0 + c < dim) {
+      if (e0 + c < vdim) {
         float sum = 0.f;
 #pragma unroll
         for (int x = 0; x < GROUPS; ++x) sum += part_s[t][x][c];
-        out[(size_t)(first + t0 + t) * heads * dim + col0 + e0 + c] = sum;
+        out[(size_t)(first + t0 + t) * heads * vdim + vcol0 + e0 + c] = AFTER ? sum * scale : sum;
       }
     }
   }
 #pragma unroll
   for (int x = 0; x < DPT; ++x) {
     const int d = d0 + x;
-    if (d < dim && e < dim) mine[(size_t)d * dim + e] = s[x];
+    if (d < dim && e < vdim) mine[(size_t)d * vdim + e] = s[x];
   }
 }
 
-template <int DPT, int COLS>
+template <int DPT, int COLS, bool AFTER>
 int launch_scan(const float* r, long r_stride, const float* k, long k_stride, const float* v, long v_stride, const float* w,
                 const float* u, float* out, float* state, long state_stride, const int* cu_q, const int* state_slots, int n_seqs,
-                int heads, int dim, cudaStream_t stream) {
-  dim3 grid((dim + COLS - 1) / COLS, heads, n_seqs);
+                int heads, int dim, int vdim, float scale, cudaStream_t stream) {
+  dim3 grid((vdim + COLS - 1) / COLS, heads, n_seqs);
   constexpr int GROUPS = RANGES * (32 / COLS);
   constexpr size_t smem = (size_t)(2 * 3 * CHUNK * GROUPS * DPT + 2 * CHUNK * COLS + CHUNK * GROUPS * COLS) * sizeof(float);
   static LbPerDeviceOnce once;
   if (smem > 48 * 1024 && once.first()) {
-    cudaFuncSetAttribute(wkv_scan_kernel<DPT, COLS, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    cudaFuncSetAttribute(wkv_scan_kernel<DPT, COLS, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    cudaFuncSetAttribute(wkv_scan_kernel<DPT, COLS, true, AFTER>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    cudaFuncSetAttribute(wkv_scan_kernel<DPT, COLS, false, AFTER>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   }
   const bool vec = dim % 4 == 0 && r_stride % 4 == 0 && k_stride % 4 == 0 && (uintptr_t)r % 16 == 0 && (uintptr_t)k % 16 == 0 &&
                    (uintptr_t)w % 16 == 0;
-  if (vec) lb_launch(wkv_scan_kernel<DPT, COLS, true>, grid, SCAN_THREADS, smem, stream, r, r_stride, k, k_stride, v, v_stride, w, u, out, state,
-                     state_stride, cu_q, state_slots, heads, dim);
-  else lb_launch(wkv_scan_kernel<DPT, COLS, false>, grid, SCAN_THREADS, smem, stream, r, r_stride, k, k_stride, v, v_stride, w, u, out, state,
-                 state_stride, cu_q, state_slots, heads, dim);
+  if (vec) lb_launch(wkv_scan_kernel<DPT, COLS, true, AFTER>, grid, SCAN_THREADS, smem, stream, r, r_stride, k, k_stride, v, v_stride, w, u, out, state,
+                     state_stride, cu_q, state_slots, heads, dim, vdim, scale);
+  else lb_launch(wkv_scan_kernel<DPT, COLS, false, AFTER>, grid, SCAN_THREADS, smem, stream, r, r_stride, k, k_stride, v, v_stride, w, u, out, state,
+                 state_stride, cu_q, state_slots, heads, dim, vdim, scale);
   return lb_last_error();
 }
 }  // namespace
@@ -330,24 +350,40 @@ LB_EXPORT int lb_wkv_shift_mix(int dtype, const void* h, const float* mu, float*
   return lb_last_error();
 }
 
-// a float [T, a_stride] (the first `rank` columns); w2 [channels, rank] in the run's type; w0 float [channels]; decay float [T, channels].
-LB_EXPORT int lb_wkv_decay(int dtype, const float* a, long a_stride, const void* w2, const float* w0, float* decay, int tokens,
-                           int channels, int rank, cudaStream_t stream) {
+namespace {
+template <bool GATE>
+int launch_decay(int dtype, const float* a, long a_stride, const void* w2, const float* w0, float* decay, int tokens, int channels,
+                 int rank, float inv_tau, cudaStream_t stream) {
   if (tokens <= 0) return 0;
   const size_t smem = (size_t)DECAY_TOKENS * ((rank + 3) & ~3) * sizeof(float);
   if (channels <= 0 || rank <= 0 || smem > 48 * 1024) return LB_ERR_SIZE;
   dim3 grid((tokens + DECAY_TOKENS - 1) / DECAY_TOKENS, (channels + 255) / 256);
   const bool vec = rank % 4 == 0 && (uintptr_t)w2 % 16 == 0;
+#define LB_DECAY(T, V) lb_launch(wkv_decay_kernel<T, V, GATE>, grid, 256, smem, stream, a, a_stride, (const T*)w2, w0, decay, tokens, channels, rank, inv_tau)
   if (dtype == LB_F32) {
-    if (vec) lb_launch(wkv_decay_kernel<float, true>, grid, 256, smem, stream, a, a_stride, (const float*)w2, w0, decay, tokens, channels, rank);
-    else lb_launch(wkv_decay_kernel<float, false>, grid, 256, smem, stream, a, a_stride, (const float*)w2, w0, decay, tokens, channels, rank);
+    if (vec) LB_DECAY(float, true); else LB_DECAY(float, false);
   } else if (dtype == LB_BF16) {
-    if (vec) lb_launch(wkv_decay_kernel<bf16, true>, grid, 256, smem, stream, a, a_stride, (const bf16*)w2, w0, decay, tokens, channels, rank);
-    else lb_launch(wkv_decay_kernel<bf16, false>, grid, 256, smem, stream, a, a_stride, (const bf16*)w2, w0, decay, tokens, channels, rank);
+    if (vec) LB_DECAY(bf16, true); else LB_DECAY(bf16, false);
   } else {
     return LB_ERR_DTYPE;
   }
+#undef LB_DECAY
   return lb_last_error();
+}
+}  // namespace
+
+// a float [T, a_stride] (the first `rank` columns); w2 [channels, rank] in the run's type; w0 float [channels]; decay float
+// [T, channels] = exp(-exp(w0 + W2 tanh(a))).
+LB_EXPORT int lb_wkv_decay(int dtype, const float* a, long a_stride, const void* w2, const float* w0, float* decay, int tokens,
+                           int channels, int rank, cudaStream_t stream) {
+  return launch_decay<false>(dtype, a, a_stride, w2, w0, decay, tokens, channels, rank, 1.f, stream);
+}
+
+// The same shapes; decay = sigmoid(w0 + W2 a)^(1 / tau).
+LB_EXPORT int lb_gate_decay(int dtype, const float* a, long a_stride, const void* w2, const float* w0, float* decay, int tokens,
+                            int channels, int rank, float tau, cudaStream_t stream) {
+  if (!(tau > 0.f)) return LB_ERR_SIZE;
+  return launch_decay<true>(dtype, a, a_stride, w2, w0, decay, tokens, channels, rank, 1.0f / tau, stream);
 }
 
 // S of head h of a request at state[slot * state_stride + h * dim * dim].
@@ -356,7 +392,7 @@ LB_EXPORT int lb_wkv_scan(const float* r, long r_stride, const float* k, long k_
                           const int* state_slots, int n_seqs, int heads, int dim, cudaStream_t stream) {
   if (n_seqs <= 0) return 0;
   if (heads <= 0 || heads > 65535 || n_seqs > 65535 || dim <= 0 || dim > 256) return LB_ERR_SIZE;
-#define LB_WKV(DPT, COLS) launch_scan<DPT, COLS>(r, r_stride, k, k_stride, v, v_stride, w, u, out, state, state_stride, cu_q, state_slots, n_seqs, heads, dim, stream)
+#define LB_WKV(DPT, COLS) launch_scan<DPT, COLS, false>(r, r_stride, k, k_stride, v, v_stride, w, u, out, state, state_stride, cu_q, state_slots, n_seqs, heads, dim, dim, 1.f, stream)
   // the split of S over lanes and warps is a function of the head size alone
   if (dim <= 32) return LB_WKV(4, 32);
   if (dim <= 64) return LB_WKV(4, 16);
@@ -364,4 +400,19 @@ LB_EXPORT int lb_wkv_scan(const float* r, long r_stride, const float* k, long k_
   if (dim <= 192) return LB_WKV(12, 16);
   return LB_WKV(16, 16);
 #undef LB_WKV
+}
+
+// Gated linear attention: S of head h of a request at state[slot * state_stride + h * dim * vdim].
+LB_EXPORT int lb_gated_scan(const float* q, long q_stride, const float* k, long k_stride, const float* v, long v_stride,
+                            const float* w, float* out, float* state, long state_stride, const int* cu_q,
+                            const int* state_slots, int n_seqs, int heads, int dim, int vdim, float scale, cudaStream_t stream) {
+  if (n_seqs <= 0) return 0;
+  if (heads <= 0 || heads > 65535 || n_seqs > 65535 || dim <= 0 || dim > 256 || vdim <= 0) return LB_ERR_SIZE;
+#define LB_GATED(DPT, COLS) launch_scan<DPT, COLS, true>(q, q_stride, k, k_stride, v, v_stride, w, nullptr, out, state, state_stride, cu_q, state_slots, n_seqs, heads, dim, vdim, scale, stream)
+  if (dim <= 32) return LB_GATED(4, 32);
+  if (dim <= 64) return LB_GATED(4, 16);
+  if (dim <= 128) return LB_GATED(8, 16);
+  if (dim <= 192) return LB_GATED(12, 16);
+  return LB_GATED(16, 16);
+#undef LB_GATED
 }

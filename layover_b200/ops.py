@@ -63,6 +63,14 @@ def _need(t: torch.Tensor, dtype: torch.dtype | None, name: str) -> None:
         raise ValueError(f"{name} must be contiguous")
 
 
+def _need_rows(t: torch.Tensor, dtype: torch.dtype | None, name: str) -> None:
+    """A 2-D tensor with dense rows, which may be part of wider ones."""
+    if dtype is not None and t.dtype != dtype:
+        raise ValueError(f"{name} must be {dtype}, got {t.dtype}")
+    if t.dim() != 2 or t.stride(1) != 1:
+        raise ValueError(f"{name} must be 2-D with dense rows")
+
+
 _signatures_done: set[str] = set()
 
 
@@ -257,20 +265,22 @@ def swiglu(gate_up: torch.Tensor, out: torch.Tensor, block: int = 0) -> torch.Te
     return out
 
 
-GATE_ACTIVATIONS = {"silu": 0, "relu": 1, "gelu_tanh": 2}
+GATE_ACTIVATIONS = {"silu": 0, "relu": 1, "gelu_tanh": 2, "clipped_swiglu": 3}
 
 
-def gated_act(gate_up: torch.Tensor, out: torch.Tensor, activation: str, block: int = 0) -> torch.Tensor:
-    """out = act(gate) * up with act "silu", "relu" or "gelu_tanh"; layouts as `swiglu`."""
+def gated_act(gate_up: torch.Tensor, out: torch.Tensor, activation: str, block: int = 0, limit: float = 0.0,
+              slope: float = 1.0) -> torch.Tensor:
+    """out = act(gate) * up with act "silu", "relu" or "gelu_tanh", or, with "clipped_swiglu", g * sigmoid(slope g) * (u + 1)
+    where g is the gate at most `limit` and u is up within +- limit; layouts as `swiglu`."""
     _need(gate_up, None, "gate_up"); _need(out, gate_up.dtype, "out")
     inter = gate_up.shape[1] // 2
     if gate_up.shape[1] != 2 * inter or out.shape[1] != inter or out.shape[0] != gate_up.shape[0]:
         raise ValueError("gated_act: shapes do not agree")
     if activation not in GATE_ACTIVATIONS:
         raise ValueError(f"gated_act: unknown activation {activation!r}")
-    fn = _fn("elementwise", "lb_gated_act", [c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p])
+    fn = _fn("elementwise", "lb_gated_act", [c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_float, c_void_p])
     _check(fn(dtype_code(gate_up.dtype), _ptr(gate_up), _ptr(out), gate_up.shape[0], inter, int(block),
-              GATE_ACTIVATIONS[activation], _stream()), "gated_act")
+              GATE_ACTIVATIONS[activation], float(limit), float(slope), _stream()), "gated_act")
     return out
 
 
@@ -317,7 +327,8 @@ def heads_bias_rope_kv(proj: torch.Tensor, q_out: torch.Tensor, k_pool: torch.Te
                        table: torch.Tensor | None, slot_map: torch.Tensor, first_v: torch.Tensor | None, blend: int,
                        blend_weight: torch.Tensor | None, q_heads: int, kv_heads: int, dim: int, vdim: int,
                        page_tokens: int, q_norm_w: torch.Tensor | None = None, k_norm_w: torch.Tensor | None = None,
-                       norm_eps: float = 0.0, neighbours: bool = False, values_from_keys: bool = False) -> None:
+                       norm_eps: float = 0.0, neighbours: bool = False, values_from_keys: bool = False,
+                       temperature: tuple[float, int] | None = None, positions: torch.Tensor | None = None) -> None:
     """Biases, a rotation of the first channels of every q and k head, an optional blend of the values with an
     earlier layer's, q to q_out and k, v to their pages.
 
@@ -329,7 +340,8 @@ def heads_bias_rope_kv(proj: torch.Tensor, q_out: torch.Tensor, k_pool: torch.Te
     q_norm_w / k_norm_w float32 [dim] (each may be None): every q (k) head is RMS-normed over its `dim` channels with that
     weight and `norm_eps`, after the biases and before the rotation. `neighbours`: channels 2i and 2i + 1 turn together
     (i < n_freq) instead of i and i + n_freq. `values_from_keys`: the row holds no values; a value head is its key head as
-    projected (with the key's bias), before norm and rotation, so vdim = dim."""
+    projected (with the key's bias), before norm and rotation, so vdim = dim. `temperature` = (coef, every): q is also
+    multiplied by 1 + coef ln(floor((p + 1) / every) + 1) at position p = positions[t] (int32 [T])."""
     _need(proj, torch.float32, "proj"); _need(k_pool, q_out.dtype, "k_pool"); _need(v_pool, q_out.dtype, "v_pool")
     _need(q_out, None, "q_out"); _need(slot_map, torch.int32, "slot_map")
     tokens = proj.shape[0]
@@ -368,14 +380,19 @@ def heads_bias_rope_kv(proj: torch.Tensor, q_out: torch.Tensor, k_pool: torch.Te
             _need(t, torch.float32, name)
             if t.numel() != dim:
                 raise ValueError(f"heads_bias_rope_kv: {name} must have {dim} entries")
+    coef, every = (float(temperature[0]), int(temperature[1])) if temperature is not None else (0.0, 0)
+    if temperature is not None:
+        _need(positions, torch.int32, "positions")
+        if positions.shape[0] != tokens or every < 1:
+            raise ValueError("heads_bias_rope_kv: a temperature needs every >= 1 and one position per token")
     fn = _fn("elementwise", "lb_heads_bias_rope_kv",
              [c_int, c_void_p, c_long] + [c_void_p] * 7 + [c_int, c_void_p, c_void_p, c_int, c_void_p] + [c_int] * 9
-             + [c_void_p, c_void_p, c_float, c_int, c_void_p])
+             + [c_void_p, c_void_p, c_float, c_int, c_void_p, c_float, c_int, c_void_p])
     _check(fn(dtype_code(q_out.dtype), _ptr(proj), proj.stride(0), _ptr(q_out), _ptr(k_pool), _ptr(v_pool), _ptr(q_bias),
               _ptr(k_bias), _ptr(v_bias), _ptr(table), n_freq, _ptr(slot_map), _ptr(first_v if blend else None), int(blend),
               _ptr(blend_weight if blend == 2 else None), tokens, q_heads, kv_heads, dim, vdim, page_tokens, q_room, k_room,
               v_room, _ptr(q_norm_w), _ptr(k_norm_w), float(norm_eps), (1 if neighbours else 0) | (2 if values_from_keys else 0),
-              _stream()), "heads_bias_rope_kv")
+              _ptr(positions if every else None), coef, every, _stream()), "heads_bias_rope_kv")
 
 
 def channel_gate(heads: torch.Tensor, logits: torch.Tensor, out: torch.Tensor, q_heads: int, vdim: int) -> torch.Tensor:
@@ -416,10 +433,11 @@ def softcap(logits: torch.Tensor, cap: float) -> torch.Tensor:
 
 
 # ------------------------------------------------------------------ routed experts
-EXPERT_ACTIVATIONS = {"silu": 0, "relu": 1, "relu2": 2}
+EXPERT_ACTIVATIONS = {"silu": 0, "relu": 1, "relu2": 2, "clipped_swiglu": 3}
+ROUTE_SCORES = {"sigmoid": 0, "softmax": 1}     # of a chosen expert's logit alone, or over the chosen logits
 
 
-def _route_options(experts: int, correction, groups, keep_groups, renormalize, route_scale, what: str):
+def _route_options(experts: int, correction, groups, keep_groups, renormalize, route_scale, score, what: str):
     """The router's further options as the kernels take them (see `moe_route`)."""
     groups = int(groups or 0)
     keep = int(keep_groups or groups or 0)
@@ -431,20 +449,25 @@ def _route_options(experts: int, correction, groups, keep_groups, renormalize, r
         raise ValueError(f"{what}: the experts must form equal groups of which 1..groups are kept")
     if not float(route_scale) > 0:
         raise ValueError(f"{what}: route_scale must be positive")
-    return [_ptr(correction), groups, keep, int(bool(renormalize)), float(route_scale)]
+    if score not in ROUTE_SCORES:
+        raise ValueError(f"{what}: unknown score {score!r}")
+    if score == "softmax" and (correction is not None or groups > 1 or renormalize or float(route_scale) != 1.0):
+        raise ValueError(f"{what}: softmax weights do not combine with corrections, groups, renormalisation or a scale")
+    return [_ptr(correction), groups, keep, int(bool(renormalize)), float(route_scale), ROUTE_SCORES[score]]
 
 
 def moe_route(h: torch.Tensor, router: torch.Tensor, top: int, ids: torch.Tensor, scores: torch.Tensor,
               shared_w: torch.Tensor | None = None, shared_factor: torch.Tensor | None = None,
               correction: torch.Tensor | None = None, groups: int | None = None, keep_groups: int | None = None,
-              renormalize: bool = False, route_scale: float = 1.0) -> None:
+              renormalize: bool = False, route_scale: float = 1.0, score: str = "sigmoid") -> None:
     """ids[t, k], scores[t, k]: the `top` experts with the largest router logits of token t (ties: the lower index) and
     sigmoid of those logits. h [T, H] in the run's type; router float32 [experts, H]; logits are 32-bit dot products.
     `shared_w` float32 [H]: also shared_factor[t] = sigmoid(shared_w . h[t]).
     `correction` float32 [experts]: the choice is made on sigmoid + correction, the scores stay the sigmoids. `groups` > 1:
     the experts form that many equal groups of neighbours, a group's score is the sum of its two largest choice scores,
     and only experts of the `keep_groups` best groups can be chosen. `renormalize`: the chosen scores are divided by their
-    sum (+ 1e-20); `route_scale` then multiplies them."""
+    sum (+ 1e-20); `route_scale` then multiplies them. `score` "softmax": the scores are the softmax over the chosen logits
+    (and none of the further options apply)."""
     _need(h, None, "h"); _need(router, torch.float32, "router"); _need(ids, torch.int32, "ids"); _need(scores, torch.float32, "scores")
     tokens, hidden = h.shape
     experts = router.shape[0]
@@ -454,15 +477,15 @@ def moe_route(h: torch.Tensor, router: torch.Tensor, top: int, ids: torch.Tensor
         _need(shared_w, torch.float32, "shared_w"); _need(shared_factor, torch.float32, "shared_factor")
         if shared_w.numel() != hidden or shared_factor.numel() != tokens:
             raise ValueError("moe_route: shared_w [H] and shared_factor [T]")
-    options = _route_options(experts, correction, groups, keep_groups, renormalize, route_scale, "moe_route")
-    fn = _fn("moe", "lb_moe_route", [c_int] + [c_void_p] * 6 + [c_int] * 4 + [c_void_p, c_int, c_int, c_int, c_float, c_void_p])
+    options = _route_options(experts, correction, groups, keep_groups, renormalize, route_scale, score, "moe_route")
+    fn = _fn("moe", "lb_moe_route", [c_int] + [c_void_p] * 6 + [c_int] * 4 + [c_void_p, c_int, c_int, c_int, c_float, c_int, c_void_p])
     _check(fn(dtype_code(h.dtype), _ptr(h), _ptr(router), _ptr(shared_w), _ptr(ids), _ptr(scores), _ptr(shared_factor), tokens,
               hidden, experts, int(top), *options, _stream()), "moe_route")
 
 
 def moe_select(logits: torch.Tensor, experts: int, top: int, ids: torch.Tensor, scores: torch.Tensor,
                shared_factor: torch.Tensor | None = None, correction: torch.Tensor | None = None, groups: int | None = None,
-               keep_groups: int | None = None, renormalize: bool = False, route_scale: float = 1.0) -> None:
+               keep_groups: int | None = None, renormalize: bool = False, route_scale: float = 1.0, score: str = "sigmoid") -> None:
     """What `moe_route` chooses, from router logits that a matrix product left in float32 [T, >= experts (+ 1)]: the
     `top` largest of the first `experts` columns (ties: the lower index), their sigmoids, and, with `shared_factor`,
     sigmoid of column `experts`."""
@@ -473,9 +496,9 @@ def moe_select(logits: torch.Tensor, experts: int, top: int, ids: torch.Tensor, 
         raise ValueError("moe_select: shapes do not agree")
     if shared_factor is not None:
         _need(shared_factor, torch.float32, "shared_factor")
-    options = _route_options(experts, correction, groups, keep_groups, renormalize, route_scale, "moe_select")
+    options = _route_options(experts, correction, groups, keep_groups, renormalize, route_scale, score, "moe_select")
     fn = _fn("moe", "lb_moe_select", [c_void_p, c_long, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
-                                      c_void_p, c_int, c_int, c_int, c_float, c_void_p])
+                                      c_void_p, c_int, c_int, c_int, c_float, c_int, c_void_p])
     _check(fn(_ptr(logits), logits.stride(0), _ptr(ids), _ptr(scores), _ptr(shared_factor), tokens, int(experts), int(top),
               *options, _stream()), "moe_select")
 
@@ -492,11 +515,12 @@ def moe_group(ids: torch.Tensor, experts: int, offsets: torch.Tensor, order: tor
 
 def moe_expert_up(h: torch.Tensor, order: torch.Tensor, offsets: torch.Tensor, scores: torch.Tensor | None,
                   gate_up: torch.Tensor, act: torch.Tensor, top: int, activation: str = "silu",
-                  interleaved: bool = False, gated: bool = True) -> torch.Tensor:
+                  interleaved: bool = False, gated: bool = True, limit: float = 0.0, slope: float = 1.0) -> torch.Tensor:
     """act[place] = act_fn(s * gate_e h[token]) * (s * up_e h[token]) for every place of `order` (pair = token * top + k, s =
     scores[pair] or 1): gate_up [experts, 2 * inter, H] (gate rows, then up rows; `interleaved`: every expert's rows in
     `interleave_gate_up`'s layout), act [pairs, inter] in the run's type. `gated` False: experts without a gate, gate_up
-    [experts, inter, H] and act[place] = relu(up_e h[token])^2 (activation "relu2", no scores)."""
+    [experts, inter, H] and act[place] = relu(up_e h[token])^2 (activation "relu2", no scores). Activation
+    "clipped_swiglu" takes `limit` and `slope` as `gated_act` does."""
     _need(h, None, "h"); _need(gate_up, h.dtype, "gate_up"); _need(act, h.dtype, "act")
     experts, rows, hidden = gate_up.shape
     pairs = order.numel()
@@ -504,10 +528,10 @@ def moe_expert_up(h: torch.Tensor, order: torch.Tensor, offsets: torch.Tensor, s
     if hidden != h.shape[1] or (gated and rows % 2) or tuple(act.shape) != (pairs, inter) or pairs != h.shape[0] * top \
             or activation not in EXPERT_ACTIVATIONS or (not gated and (activation != "relu2" or interleaved or scores is not None)):
         raise ValueError("moe_expert_up: shapes do not agree")
-    fn = _fn("moe", "lb_moe_expert_up", [c_int, c_void_p, c_long] + [c_void_p] * 5 + [c_int] * 8 + [c_void_p])
+    fn = _fn("moe", "lb_moe_expert_up", [c_int, c_void_p, c_long] + [c_void_p] * 5 + [c_int] * 8 + [c_float, c_float, c_void_p])
     _check(fn(dtype_code(h.dtype), _ptr(h), h.stride(0), _ptr(order), _ptr(offsets), _ptr(scores), _ptr(gate_up), _ptr(act),
               pairs, int(top), experts, hidden, inter, EXPERT_ACTIVATIONS[activation], int(bool(interleaved)), int(bool(gated)),
-              _stream()), "moe_expert_up")
+              float(limit), float(slope), _stream()), "moe_expert_up")
     return act
 
 
@@ -589,33 +613,37 @@ def moe_scatter_rows(h: torch.Tensor, place_of: torch.Tensor, scale: torch.Tenso
     return rows
 
 
+GROUPED_EPILOGUES = {None: 0, "swiglu": 1, "clipped_swiglu": 3}
+
+
 def gemm_tcgen05_grouped(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, tile_rows: torch.Tensor, groups: int,
-                         epilogue: str | None = None) -> torch.Tensor:
+                         epilogue: str | None = None, limit: float = 0.0, slope: float = 1.0) -> torch.Tensor:
     """out[M, N] = a[M, K] @ w_g[N, K]^T tile by tile: every tile of 128 rows of `a` is multiplied by the weights of ONE
     group, the [N, K] matrix that begins at row tile_rows[tile] of w [groups * N, K]; tile_rows [M / 128 + 1] ends with the
     number of tiles in use (all at the front; the others are skipped). It is int32 on the device, written by an earlier kernel. M is a multiple of 128. epilogue "swiglu" as in
-    `gemm_tcgen05` (each group's rows interleaved by `interleave_gate_up`)."""
+    `gemm_tcgen05` (each group's rows interleaved by `interleave_gate_up`), "clipped_swiglu" the same with that activation
+    (see `gated_act`)."""
     if a.dtype != torch.bfloat16 or w.dtype != torch.bfloat16 or a.dim() != 2 or w.dim() != 2:
         raise ValueError("gemm_tcgen05_grouped: operands must be 2-D bfloat16")
     m, k = a.shape
     if w.shape[0] % groups or w.shape[1] != k or m % MOE_TILE_ROWS:
         raise ValueError("gemm_tcgen05_grouped: shapes do not agree")
     n = w.shape[0] // groups
-    if epilogue not in (None, "swiglu"):
+    if epilogue not in GROUPED_EPILOGUES:
         raise ValueError(f"gemm_tcgen05_grouped: unknown epilogue {epilogue!r}")
-    out_cols = n // 2 if epilogue == "swiglu" else n
-    if epilogue == "swiglu" and (n % (2 * SWIGLU_BLOCK) or out.dtype != torch.bfloat16):
-        raise ValueError("gemm_tcgen05_grouped: the swiglu epilogue needs interleaved weights and a bfloat16 output")
+    out_cols = n // 2 if epilogue else n
+    if epilogue and (n % (2 * SWIGLU_BLOCK) or out.dtype != torch.bfloat16):
+        raise ValueError("gemm_tcgen05_grouped: a gated epilogue needs interleaved weights and a bfloat16 output")
     _need(tile_rows, torch.int32, "tile_rows")
     if tuple(out.shape) != (m, out_cols) or out.stride(1) != 1 or tile_rows.numel() != m // MOE_TILE_ROWS + 1:
         raise ValueError("gemm_tcgen05_grouped: out [M, N], one tile entry per 128 rows and the count of tiles in use behind them")
     partials, counters, sms = gemm_scratch(a.device)
     fn = _fn("gemm_tcgen05", "lb_gemm_tcgen05_grouped",
              [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_long, c_long, c_long, c_void_p, c_void_p, c_long,
-              c_void_p, c_int, c_int, c_int, c_void_p])
+              c_void_p, c_int, c_int, c_int, c_float, c_float, c_void_p])
     _check(fn(_ptr(a), _ptr(w), _ptr(out), dtype_code(out.dtype), m, n, k, int(groups), a.stride(0), w.stride(0), out.stride(0),
               _ptr(tile_rows), _ptr(partials), partials.numel(), _ptr(counters), counters.numel(), sms,
-              1 if epilogue == "swiglu" else 0, _stream()), "gemm_tcgen05_grouped")
+              GROUPED_EPILOGUES[epilogue], float(limit), float(slope), _stream()), "gemm_tcgen05_grouped")
     return out
 
 
@@ -860,17 +888,19 @@ def head_gated_rmsnorm(o: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor
                        vdim: int) -> torch.Tensor:
     """out[t, h] = o[t, h] * rsqrt(mean(o[t, h]^2) + eps) * weight * silu(gate[t, h]) per head: o float32 [T, heads * vdim],
     gate float32 [T, heads * vdim] (a view into wider rows is fine), weight float32 [vdim] (shared by the heads) or
-    [heads * vdim] (a weight per channel), out in the run's type."""
-    _need(o, torch.float32, "o"); _need(weight, torch.float32, "weight"); _need(out, None, "out")
+    [heads * vdim] (a weight per channel), out in the run's type (a view into wider rows is fine)."""
+    _need(o, torch.float32, "o"); _need(weight, torch.float32, "weight")
+    if out.dim() != 2 or out.stride(1) != 1:
+        raise ValueError("head_gated_rmsnorm: out must have dense rows")
     tokens = o.shape[0]
     if gate.dtype != torch.float32 or tuple(o.shape) != (tokens, heads * vdim) or tuple(out.shape) != (tokens, heads * vdim) or gate.dim() != 2 \
             or gate.stride(1) != 1 or tuple(gate.shape) != (tokens, heads * vdim) or weight.numel() not in (vdim, heads * vdim):
         raise ValueError("head_gated_rmsnorm: shapes do not agree")
     per_channel = weight.numel() == heads * vdim and heads > 1
     fn = _fn("delta_rule", "lb_head_gated_rmsnorm", [c_int, c_void_p, c_void_p, c_long, c_void_p, c_void_p, c_int, c_int, c_int,
-                                                     c_float, c_int, c_void_p])
+                                                     c_float, c_int, c_long, c_void_p])
     _check(fn(dtype_code(out.dtype), _ptr(o), _ptr(gate), gate.stride(0), _ptr(weight), _ptr(out), tokens, heads, vdim, float(eps),
-              vdim if per_channel else 0, _stream()), "head_gated_rmsnorm")
+              vdim if per_channel else 0, out.stride(0), _stream()), "head_gated_rmsnorm")
     return out
 
 
@@ -936,6 +966,41 @@ def wkv_scan(r: torch.Tensor, k: torch.Tensor, v: torch.Tensor, w: torch.Tensor,
     return out
 
 
+def gate_decay(a: torch.Tensor, w2: torch.Tensor, w0: torch.Tensor, tau: float, decay: torch.Tensor) -> torch.Tensor:
+    """decay[t, c] = sigmoid(w0[c] + sum_j w2[c, j] a[t, j])^(1 / tau) in 32-bit; tensors as `wkv_decay`."""
+    _need(w2, None, "w2"); _need(w0, torch.float32, "w0"); _need(decay, torch.float32, "decay")
+    channels, rank = w2.shape
+    tokens = a.shape[0]
+    if a.dtype != torch.float32 or a.dim() != 2 or a.stride(1) != 1 or a.shape[1] < rank or w0.numel() != channels \
+            or tuple(decay.shape) != (tokens, channels) or not tau > 0:
+        raise ValueError("gate_decay: shapes do not agree, or tau is not positive")
+    fn = _fn("wkv", "lb_gate_decay", [c_int, c_void_p, c_long, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_void_p])
+    _check(fn(dtype_code(w2.dtype), _ptr(a), a.stride(0), _ptr(w2), _ptr(w0), _ptr(decay), tokens, channels, rank, float(tau),
+              _stream()), "gate_decay")
+    return decay
+
+
+def gated_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, w: torch.Tensor, out: torch.Tensor, state: torch.Tensor, batch,
+               heads: int, dim: int, vdim: int, scale: float) -> torch.Tensor:
+    """Gated linear attention over every sequence's tokens of the step, from and into the requests' state slots:
+    S <- diag(w_t) S + k_t v_t^T, then o_t = scale * S^T q_t. q, k float32 [T, heads * dim], v float32 [T, heads * vdim]
+    (views into wider rows are fine), w float32 [T, heads * dim], out float32 [T, heads * vdim], state float32
+    [slots, heads, dim, vdim]."""
+    for name, t in (("w", w), ("out", out), ("state", state)):
+        _need(t, torch.float32, name)
+    tokens = out.shape[0]
+    for name, t, n in (("q", q, heads * dim), ("k", k, heads * dim), ("v", v, heads * vdim)):
+        if t.dtype != torch.float32 or t.dim() != 2 or t.stride(1) != 1 or tuple(t.shape) != (tokens, n):
+            raise ValueError(f"gated_scan: {name} must be float32 [tokens, {n}] with dense rows")
+    if out.shape[1] != heads * vdim or tuple(w.shape) != (tokens, heads * dim) or tuple(state.shape[1:]) != (heads, dim, vdim):
+        raise ValueError("gated_scan: shapes do not agree")
+    fn = _fn("wkv", "lb_gated_scan", [c_void_p, c_long, c_void_p, c_long, c_void_p, c_long, c_void_p, c_void_p, c_void_p, c_long,
+                                      c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_void_p])
+    _check(fn(_ptr(q), q.stride(0), _ptr(k), k.stride(0), _ptr(v), v.stride(0), _ptr(w), _ptr(out), _ptr(state), state.stride(0),
+              _ptr(batch.cu_q), _ptr(batch.state_slots), batch.n_seqs, heads, dim, vdim, float(scale), _stream()), "gated_scan")
+    return out
+
+
 # ------------------------------------------------------------------ matrix products
 def gemm_simt(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
     """out[M, N] = a[M, K] @ w[N, K]^T with 32-bit FFMA accumulation (no tensor cores).
@@ -970,7 +1035,8 @@ def attention_simt(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, 
                    block_table: torch.Tensor, cu_q: torch.Tensor, ctx_len: torch.Tensor, tile_seq: torch.Tensor,
                    tile_q0: torch.Tensor, n_tiles: int, q_heads: int, kv_heads: int, dim: int, page_tokens: int,
                    scale: float, window: int = 0, vdim: int | None = None, sinks: torch.Tensor | None = None,
-                   gates: torch.Tensor | None = None, chunk: int = 0, keep_first: int = 0) -> torch.Tensor:
+                   gates: torch.Tensor | None = None, chunk: int = 0, keep_first: int = 0, softcap: float = 0.0,
+                   out_scale: float = 1.0) -> torch.Tensor:
     """Paged causal attention in 32-bit arithmetic for any mix of segment lengths.
 
     q [T, q_heads * dim]; out [T, q_heads * vdim] (vdim defaults to dim); pools [pages, kv_heads, page_tokens,
@@ -978,9 +1044,10 @@ def attention_simt(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, 
     [n_tiles] list the query tiles. `sinks` float32 [q_heads]: a score per head that joins the softmax's
     denominator only; `gates` float32 [T, q_heads]: a factor on each head's output. `chunk` > 0: a query sees
     only the keys of its own chunk of that many positions (counted from position 0 of its sequence). `keep_first` > 0:
-    behind a window the first `keep_first` keys of the sequence stay visible."""
+    behind a window the first `keep_first` keys of the sequence stay visible. `softcap` > 0: a score s becomes softcap *
+    tanh(s / softcap). `out_scale` multiplies the outputs; `out` may be a view into wider rows."""
     vdim = dim if vdim is None else int(vdim)
-    _need(q, None, "q"); _need(out, q.dtype, "out"); _need(k_pool, q.dtype, "k_pool"); _need(v_pool, q.dtype, "v_pool")
+    _need(q, None, "q"); _need_rows(out, q.dtype, "out"); _need(k_pool, q.dtype, "k_pool"); _need(v_pool, q.dtype, "v_pool")
     if tuple(out.shape) != (q.shape[0], q_heads * vdim) or k_pool.shape[-1] != dim or v_pool.shape[-1] != vdim:
         raise ValueError("attention_simt: out or the pools do not match the head sizes")
     if sinks is not None:
@@ -996,22 +1063,23 @@ def attention_simt(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, 
         _need(t, torch.int32, name)
     fn = _fn("attention_simt", "lb_attention_simt",
              [c_int] + [c_void_p] * 5 + [c_int] + [c_void_p] * 4 + [c_int] * 5 + [c_float, c_int, c_int, c_void_p,
-                                                                                c_void_p, c_int, c_int, c_void_p])
+                                                                                c_void_p, c_int, c_int, c_float, c_float, c_long, c_void_p])
     _check(fn(dtype_code(q.dtype), _ptr(q), _ptr(k_pool), _ptr(v_pool), _ptr(out), _ptr(block_table),
               block_table.shape[1], _ptr(cu_q), _ptr(ctx_len), _ptr(tile_seq), _ptr(tile_q0), n_tiles, q_heads,
               kv_heads, dim, page_tokens, float(scale), int(window), vdim, _ptr(sinks), _ptr(gates), int(chunk), int(keep_first),
-              _stream()),
+              float(softcap), float(out_scale), out.stride(0), _stream()),
            "attention_simt")
     return out
 
 
 def attention_f32(q, cache, out, block_table, batch, q_heads, kv_heads, dim, page_tokens, scale, window, vdim=None,
-                  sinks=None, gates=None, chunk=0, keep_first=0):
+                  sinks=None, gates=None, chunk=0, keep_first=0, softcap=0.0, out_scale=1.0):
     """The 32-bit path's attention for one step: one kernel for every mix of segment lengths (and, in
     either precision, the attention with sinks, head gates or values of another size than keys)."""
     tiles = batch.tiles[attention_simt_block_queries()]
     attention_simt(q, cache.k_pool, cache.v_pool, out, block_table, batch.cu_q, batch.ctx_len, tiles.tile_seq, tiles.tile_q0,
-                   tiles.count, q_heads, kv_heads, dim, page_tokens, scale, window, vdim, sinks, gates, chunk, keep_first)
+                   tiles.count, q_heads, kv_heads, dim, page_tokens, scale, window, vdim, sinks, gates, chunk, keep_first,
+                   softcap, out_scale)
 
 
 # ------------------------------------------------------------------ sampling
@@ -1267,23 +1335,29 @@ def _sink_arguments(sinks, gates, tokens, q_heads, what):
 
 
 def attention_prefill_bf16(q, k_pool, v_pool, out, block_table, cu_q, ctx_len, tile_seq, tile_q0, n_tiles, q_heads,
-                           kv_heads, dim, page_tokens, scale, window=0, sinks=None, gates=None, exact_weights=False, keep_first=0):
+                           kv_heads, dim, page_tokens, scale, window=0, sinks=None, gates=None, exact_weights=False, keep_first=0,
+                           softcap=0.0, out_scale=1.0):
     """Tensor-core paged attention for prompt portions: tiles of 64 queries, any number of queries per sequence.
     `window` > 0: the last `window` keys; `window` < 0: a chunked mask, the keys of the query's own chunk of -window positions.
     `sinks` float32 [q_heads] join the softmax's denominator only, `gates` float32 [T, q_heads] multiply the
     heads' outputs, `exact_weights` keeps 16 bits of the weights' mantissa in the second product. `keep_first` (with a
-    window): the first keys of a sequence stay visible behind the window."""
+    window): the first keys of a sequence stay visible behind the window. `softcap` > 0: a score s becomes softcap *
+    tanh(s / softcap); `out_scale` multiplies the outputs (each asks for the variant with exact weights); `out` may be a
+    view into wider rows."""
     _sink_arguments(sinks, gates, q.shape[0], q_heads, "attention_prefill_bf16")
-    for name, t in (("q", q), ("out", out), ("k_pool", k_pool), ("v_pool", v_pool)):
+    _need_rows(out, torch.bfloat16, "out")
+    for name, t in (("q", q), ("k_pool", k_pool), ("v_pool", v_pool)):
         _need(t, torch.bfloat16, name)
     for name, t in (("block_table", block_table), ("cu_q", cu_q), ("ctx_len", ctx_len), ("tile_seq", tile_seq),
                     ("tile_q0", tile_q0)):
         _need(t, torch.int32, name)
     fn = _fn("attention_mma", "lb_attention_prefill_bf16",
-             [c_void_p] * 5 + [c_int] + [c_void_p] * 4 + [c_int] * 5 + [c_float, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p])
+             [c_void_p] * 5 + [c_int] + [c_void_p] * 4 + [c_int] * 5 + [c_float, c_int, c_void_p, c_void_p, c_int, c_int, c_float, c_float,
+                                                                              c_long, c_void_p])
     _check(fn(_ptr(q), _ptr(k_pool), _ptr(v_pool), _ptr(out), _ptr(block_table), block_table.shape[1], _ptr(cu_q),
               _ptr(ctx_len), _ptr(tile_seq), _ptr(tile_q0), n_tiles, q_heads, kv_heads, dim, page_tokens, float(scale),
-              int(window), _ptr(sinks), _ptr(gates), int(bool(exact_weights)), int(keep_first), _stream()), "attention_prefill_bf16")
+              int(window), _ptr(sinks), _ptr(gates), int(bool(exact_weights)), int(keep_first), float(softcap),
+              float(out_scale), out.stride(0), _stream()), "attention_prefill_bf16")
     return out
 
 
@@ -1356,14 +1430,16 @@ def decode_splits(n_seqs: int, q_heads: int, kv_heads: int, dim: int, max_contex
 
 def attention_decode_bf16(q, k_pool, v_pool, out, block_table, cu_q, ctx_len, seq_list, n_seqs, q_heads, kv_heads, dim,
                           page_tokens, scale, window=0, splits=1, stages=3, sinks=None, gates=None, exact_weights=False,
-                          keep_first=0, kv_share=1):
+                          keep_first=0, kv_share=1, softcap=0.0, out_scale=1.0):
     """Tensor-core paged attention for sequences with one new token each, the context split `splits` ways
     (`stages` 2: the variant that fits three blocks an SM, see `decode_plan`). `sinks`, `gates` and
     `exact_weights` as in `attention_prefill_bf16` (those variants merge their splits through scratch memory). `kv_share` > 1:
     `kv_heads` counts groups of at most 16 query heads, and kv_share neighbouring groups read the same stored head (the pools
-    hold kv_heads / kv_share heads): more query heads on one key/value head than the kernel's tile has rows."""
+    hold kv_heads / kv_share heads): more query heads on one key/value head than the kernel's tile has rows. `softcap`,
+    `out_scale` and a strided `out` as in `attention_prefill_bf16`."""
     _sink_arguments(sinks, gates, q.shape[0], q_heads, "attention_decode_bf16")
-    for name, t in (("q", q), ("out", out), ("k_pool", k_pool), ("v_pool", v_pool)):
+    _need_rows(out, torch.bfloat16, "out")
+    for name, t in (("q", q), ("k_pool", k_pool), ("v_pool", v_pool)):
         _need(t, torch.bfloat16, name)
     for name, t in (("block_table", block_table), ("cu_q", cu_q), ("ctx_len", ctx_len)):
         _need(t, torch.int32, name)
@@ -1372,11 +1448,13 @@ def attention_decode_bf16(q, k_pool, v_pool, out, block_table, cu_q, ctx_len, se
     partials, counters = attention_scratch(q.device)
     fn = _fn("attention_mma", "lb_attention_decode_bf16",
              [c_void_p] * 5 + [c_int] + [c_void_p] * 3 + [c_int] * 5 + [c_float, c_int, c_int, c_void_p, c_long, c_void_p,
-                                                                        c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p])
+                                                                        c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_float,
+                                                                        c_float, c_long, c_void_p])
     _check(fn(_ptr(q), _ptr(k_pool), _ptr(v_pool), _ptr(out), _ptr(block_table), block_table.shape[1], _ptr(cu_q),
               _ptr(ctx_len), _ptr(seq_list), n_seqs, q_heads, kv_heads, dim, page_tokens, float(scale), int(window),
               int(splits), _ptr(partials), partials.numel(), _ptr(counters), counters.numel(), int(stages), _ptr(sinks),
-              _ptr(gates), int(bool(exact_weights)), int(keep_first), int(kv_share), _stream()), "attention_decode_bf16")
+              _ptr(gates), int(bool(exact_weights)), int(keep_first), int(kv_share), float(softcap), float(out_scale),
+              out.stride(0), _stream()), "attention_decode_bf16")
     return out
 
 
@@ -1437,14 +1515,15 @@ def attention_tcgen05_prefill(q, pool, layer, out, block_table, cu_q, ctx_len, t
 
 
 def attention_bf16(q, cache, out, block_table, batch, q_heads, kv_heads, dim, page_tokens, scale, window, sinks=None,
-                   gates=None, exact_weights=False, chunk=0, keep_first=0, decode_share=1):
+                   gates=None, exact_weights=False, chunk=0, keep_first=0, decode_share=1, softcap=0.0, out_scale=1.0):
     """The bfloat16 path's attention for one step: prompt portions go through the tcgen05 tile kernel
     where it takes the sizes (head size 128, pages of 8..128 tokens), else through the mma.sync
     one; single tokens, alone or beside prompt portions, go through the split decode kernel. With
     sinks, gates or exact weights the mma.sync kernels' variants for those run everywhere. `decode_share` > 1: the
     decode kernel takes the query heads of a key/value head as that many groups (each at most 16 heads)."""
-    plain = sinks is None and gates is None and not exact_weights and not chunk and not keep_first
-    extras = dict(sinks=sinks, gates=gates, exact_weights=exact_weights, keep_first=keep_first)
+    plain = sinks is None and gates is None and not exact_weights and not chunk and not keep_first and not softcap \
+        and out_scale == 1.0 and out.is_contiguous()
+    extras = dict(sinks=sinks, gates=gates, exact_weights=exact_weights, keep_first=keep_first, softcap=softcap, out_scale=out_scale)
     if chunk:
         if window:
             raise ValueError("attention_bf16: a window and a chunked mask do not combine")

@@ -64,7 +64,10 @@ class Attention(Part):
     and 2i + 1 together. Both take this path.
     `keep_first` (with `window`): the first `keep_first` tokens of a sequence stay visible behind the window, at
     their own positions; their pages stay in the cache. `exact_weights` = True asks for this path (32-bit
-    projection rows, softmax weights that keep 16 bits of mantissa in the second product) without any other option."""
+    projection rows, softmax weights that keep 16 bits of mantissa in the second product) without any other option.
+    `softcap` c: a scaled score s becomes c * tanh(s / c) before the mask. `query_temperature` = (coef, every): the query
+    at position p is multiplied by 1 + coef ln(floor((p + 1) / every) + 1), after its norm. `out_scale`: a factor on the
+    heads' outputs. These three take this path as well. A part on this path without a channel gate is `stackable`."""
 
     def __init__(self, params, prefix):
         super().__init__(params, prefix)
@@ -91,13 +94,20 @@ class Attention(Part):
         position = p.get("position")
         partial = bool(position and (int(position.params.get("rotated") or p["head_dim"]) != int(p["head_dim"])
                                      or position.kind == "rotary_pairs"))
+        self.softcap = float(p.get("softcap") or 0.0)
+        temperature = p.get("query_temperature")
+        self.temperature = (float(temperature[0]), int(temperature[1])) if temperature is not None else None
+        self.out_scale = float(p.get("out_scale", 1.0))
+        if self.softcap < 0 or (self.temperature is not None and self.temperature[1] < 1):
+            raise ValueError("attention: softcap must be positive, query_temperature (coef, every) with every >= 1")
         # biases, a partial rotation, a blend of values or a gate per channel: one kernel over 32-bit projection rows
         self.keep_first = int(p.get("keep_first") or 0)
         if self.keep_first < 0 or (self.keep_first and not p.get("window")):
             raise ValueError("attention: keep_first is a number of tokens and comes with a window")
         self.rows32 = bool(self.biases or partial or self.value_blend or (p.get("gate") and self.gate_kind == "channel")
                            or (position and (p.get("v_head_dim") or p["head_dim"]) != p["head_dim"]) or self.chunk
-                           or self.keep_first or p.get("exact_weights") or self.values_from_keys)
+                           or self.keep_first or p.get("exact_weights") or self.values_from_keys or self.softcap
+                           or self.temperature is not None or self.out_scale != 1.0)
         self.general = bool(self.vdim != self.dim or self.qk_norm == "whole" or p.get("sink") or p.get("gate") or self.rows32)
         if self.general:
             if (self.dim % 4 or self.vdim % 4) and not self.rows32:
@@ -131,7 +141,8 @@ class Attention(Part):
             wanted.append("value_blend_weight")
         self.require(*wanted)
         self.names = {k: prefix + p[k] for k in wanted}
-        self.w_qkv = self.w_o = self.q_norm_w = self.k_norm_w = self.sink = None
+        self.w_in = self.w_o = self.q_norm_w = self.k_norm_w = self.sink = None
+        self.stackable = self.rows32 and not p.get("gate")
         self._attend = self._project_heads = None
         self.room = None        # once bound: the size keys, values and queries are padded to for the tensor-core kernels
         # where the tensor-core kernels do not run: the room of a key and of a value in their pages (the 32-bit kernel
@@ -211,9 +222,9 @@ class Attention(Part):
             self._attend, self._project_heads = ops.attention_bf16, ops.gemm_qkv_heads
         n = self.names
         if self.shares_cache:
-            self.w_qkv = tensors[n["q"]]
+            self.w_in = tensors[n["q"]]
         else:
-            self.w_qkv = torch.cat((tensors.pop(n["q"]), tensors.pop(n["k"]), tensors.pop(n["v"])), dim=0).contiguous()
+            self.w_in = torch.cat((tensors.pop(n["q"]), tensors.pop(n["k"]), tensors.pop(n["v"])), dim=0).contiguous()
         self.w_o = tensors[n["o"]]
         if self.qk_norm_eps is not None:
             self.q_norm_w = tensors[n["q_norm"]]
@@ -229,7 +240,7 @@ class Attention(Part):
         used = sum(r.shape[0] for r in rows)
         if used % 16:           # whole 16-byte pieces per output row, whatever the head counts
             rows.append(torch.zeros((16 - used % 16, self.hidden), dtype=rows[0].dtype, device=rows[0].device))
-        self.w_qkv = torch.cat(rows, dim=0).contiguous()
+        self.w_in = torch.cat(rows, dim=0).contiguous()
         self.w_o = tensors[n["o"]]
         if self.qk_norm_eps is not None:
             self.q_norm_w, self.k_norm_w = tensors[n["q_norm"]], tensors[n["k_norm"]]
@@ -259,44 +270,50 @@ class Attention(Part):
         return batch.shared[key]
 
     def _forward_general(self, h, batch, cache):
-        tokens, group = h.shape[0], batch.groups[cache.group]
+        if self.rows32:
+            proj = self.runtime.linear(h, self.w_in, out_dtype=torch.float32)
+        else:
+            proj = self.runtime.linear(h, self.w_in)
+        out = torch.empty((h.shape[0], self.q_heads * (self.room or self.v_room)), dtype=h.dtype, device=h.device)
+        self.mix(proj, batch, cache, out)
+        if self.rows32 and "gate" in self.names:
+            at = self.q_heads * self.dim + self.kv_heads * (self.dim + (0 if self.values_from_keys else self.vdim))
+            gated = torch.empty((h.shape[0], self.q_heads * self.vdim), dtype=h.dtype, device=h.device)
+            out = ops.channel_gate(out, proj[:, at: at + self.q_heads * self.vdim], gated, self.q_heads, self.vdim)
+        return self.runtime.linear(out, self.w_o)
+
+    def mix(self, proj, batch, cache, out) -> None:
+        """From the stacked projection's rows to the heads' outputs, each head in its room of `out`'s rows."""
+        tokens, group = proj.shape[0], batch.groups[cache.group]
         room = self.room or self.k_room
-        q = torch.empty((tokens, self.q_heads * room), dtype=h.dtype, device=h.device)
+        q = torch.empty((tokens, self.q_heads * room), dtype=out.dtype, device=out.device)
         gates = None
         if self.rows32:
-            proj = self.runtime.linear(h, self.w_qkv, out_dtype=torch.float32)
             table = self.position.tables(batch) if self.position is not None else None
             if self.position is not None and table is None:
                 raise ValueError("attention: this position encoding offers no table for the fused kernel")
             blend = {None: 0, "keep": 1, "blend": 2}[self.value_blend]
-            kept = self._kept_values(batch, tokens, h.device) if blend else None
+            kept = self._kept_values(batch, tokens, out.device) if blend else None
             ops.heads_bias_rope_kv(proj, q, cache.k_pool, cache.v_pool, self.bias.get("q_bias"), self.bias.get("k_bias"),
                                    self.bias.get("v_bias"), table, group.slot_map, kept, blend, self.blend_weight,
                                    self.q_heads, self.kv_heads, self.dim, self.vdim, cache.page_tokens,
                                    self.q_norm_w, self.k_norm_w, float(self.qk_norm_eps or 0.0),
                                    neighbours=getattr(self.position, "pairing", "half") == "neighbours",
-                                   values_from_keys=self.values_from_keys)
+                                   values_from_keys=self.values_from_keys, temperature=self.temperature,
+                                   positions=batch.positions if self.temperature is not None else None)
         else:
-            proj = self.runtime.linear(h, self.w_qkv)
             if "gate" in self.names:
-                gates = torch.empty((tokens, self.q_heads), dtype=torch.float32, device=h.device)
+                gates = torch.empty((tokens, self.q_heads), dtype=torch.float32, device=out.device)
             ops.qk_rownorm_kv(proj, q, cache.k_pool, cache.v_pool, self.q_norm_w, self.k_norm_w, group.slot_map, gates,
                               self.q_heads, self.kv_heads, self.dim, self.vdim, cache.page_tokens, float(self.qk_norm_eps or 0.0))
         if self.room is not None:
-            out = torch.empty((tokens, self.q_heads * room), dtype=h.dtype, device=h.device)
             ops.attention_bf16(q, cache, out, group.block_table, batch, self.q_heads, self.kv_heads, room, cache.page_tokens,
                                self.scale, self.window or 0, sinks=self.sink, gates=gates, exact_weights=True, chunk=self.chunk,
-                               keep_first=self.keep_first)
+                               keep_first=self.keep_first, softcap=self.softcap, out_scale=self.out_scale)
         else:
-            out = torch.empty((tokens, self.q_heads * self.v_room), dtype=h.dtype, device=h.device)
             ops.attention_f32(q, cache, out, group.block_table, batch, self.q_heads, self.kv_heads, self.k_room, cache.page_tokens,
                               self.scale, self.window or 0, self.v_room, self.sink, gates, chunk=self.chunk,
-                              keep_first=self.keep_first)
-        if self.rows32 and "gate" in self.names:
-            at = self.q_heads * self.dim + self.kv_heads * (self.dim + (0 if self.values_from_keys else self.vdim))
-            gated = torch.empty((tokens, self.q_heads * self.vdim), dtype=h.dtype, device=h.device)
-            out = ops.channel_gate(out, proj[:, at: at + self.q_heads * self.vdim], gated, self.q_heads, self.vdim)
-        return self.runtime.linear(out, self.w_o)
+                              keep_first=self.keep_first, softcap=self.softcap, out_scale=self.out_scale)
 
     # ---- one step
     def forward(self, h: torch.Tensor, batch, cache) -> torch.Tensor:
@@ -319,10 +336,10 @@ class Attention(Part):
         k_pool, v_pool = (cache.k_pool, cache.v_pool) if own_kv else (None, None)
         heads = self._project_heads
         if (heads is not None and own_kv and table is not None and self.qk_norm_eps is not None
-                and heads(h, self.w_qkv, q, k_pool, v_pool, self.q_norm_w, self.k_norm_w, table, group.slot_map,
+                and heads(h, self.w_in, q, k_pool, v_pool, self.q_norm_w, self.k_norm_w, table, group.slot_map,
                           self.q_heads, own_kv, self.dim, cache.page_tokens, eps)):
             return q                       # projection, norm, rotation and page write were one kernel
-        qkv = self.runtime.linear(h, self.w_qkv)
+        qkv = self.runtime.linear(h, self.w_in)
         if fused:
             ops.qk_norm_rope_kv(qkv, q, k_pool, v_pool, self.q_norm_w, self.k_norm_w, table, group.slot_map,
                                 self.q_heads, own_kv, self.dim, cache.page_tokens, eps)

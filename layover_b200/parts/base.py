@@ -26,6 +26,11 @@ What each kind must offer:
   mixer           cache_need() -> PagedKVNeed | StateNeed | None, or a tuple of them (a mixer made of mixers; its
                                                       cache is then a composite view with one view per need in `parts`)
                   forward(h, batch, cache) -> [T, hidden]     cache is the view it was given for its need
+                  a mixer that can share its two products with mixers beside it has `stackable` True and, once
+                  bound, `w_in` [N, hidden], `w_o` [hidden, K] and
+                  mix(proj, batch, cache, out)                proj float32 [T, N] (w_in h) -> out [T, K] in the run's
+                                                              type, both possibly parts of wider rows; w_o is the
+                                                              caller's to apply
   feed-forward    forward(h) -> [T, hidden]
   block           forward(x, delta, batch, cache, extra=None) -> (x, delta)   the residual stream and the
                                                       not-yet-added output of the last sub-layer; extra is

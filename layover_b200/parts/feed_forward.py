@@ -13,8 +13,8 @@ from .base import Part, build_part, register_feed_forward
 class GatedMLP(Part):
     """down(act(gate(x)) * up(x)) without bias (layover/model.py:145-153); act = silu or relu.
 
-    params: hidden, inter, activation ("silu", the default, or "relu"), gate, up, down (tensor names relative to the
-    prefix). gate and up are stacked at load into one [2 inter, hidden] matrix so that one
+    params: hidden, inter, activation ("silu", the default, or one of `ops.GATE_ACTIVATIONS`; "clipped_swiglu" with
+    limit and slope), gate, up, down (tensor names relative to the prefix). gate and up are stacked at load into one [2 inter, hidden] matrix so that one
     product reads x once. In a bfloat16 run whose width allows it, the rows are interleaved for
     the tensor-core product with the activation in its epilogue and no [T, 2 inter] tensor is ever
     written; otherwise the activation kernel reads both halves of its row. The product's epilogue
@@ -27,6 +27,9 @@ class GatedMLP(Part):
         self.activation = params.get("activation", "silu")
         if self.activation not in ops.GATE_ACTIVATIONS:
             raise ValueError(f"gated_mlp: unsupported activation {self.activation!r}")
+        self._clip = dict(limit=float(params.get("limit") or 0.0), slope=float(params.get("slope", 1.0)))
+        if self.activation == "clipped_swiglu" and not self._clip["limit"] > 0:
+            raise ValueError("gated_mlp: clipped_swiglu needs a positive limit")
         self.names = {k: prefix + params[k] for k in ("gate", "up", "down")}
         self.gate_up = self.down = None
 
@@ -61,7 +64,7 @@ class GatedMLP(Part):
         gate_up = self.runtime.linear(h, self.gate_up)
         if self.activation == "silu":
             return ops.swiglu(gate_up, out, block=ops.SWIGLU_BLOCK)
-        return ops.gated_act(gate_up, out, self.activation, block=ops.SWIGLU_BLOCK)
+        return ops.gated_act(gate_up, out, self.activation, block=ops.SWIGLU_BLOCK, **self._clip)
 
     def forward(self, h: torch.Tensor) -> torch.Tensor:
         if self.fused:
@@ -71,7 +74,7 @@ class GatedMLP(Part):
         if self.activation == "silu":
             ops.swiglu(gate_up, act)
         else:
-            ops.gated_act(gate_up, act, self.activation)
+            ops.gated_act(gate_up, act, self.activation, **self._clip)
         return self.runtime.linear(act, self.down)
 
 
@@ -121,7 +124,10 @@ class RoutedExperts(Part):
     (`activation` "relu2"; there is no expert_gate tensor). The choice may be made on corrected scores (`correction`: a
     tensor of one number per expert, added to the sigmoids for the choice only), limited to the `keep_groups` best of
     `groups` equal groups of neighbouring experts (a group's score: the sum of its two largest corrected scores), and the
-    chosen scores may be divided by their sum (`renormalize`) and multiplied by `route_scale`. On the device:
+    chosen scores may be divided by their sum (`renormalize`) and multiplied by `route_scale`. `score` = "softmax": the
+    choice is made on the logits and the scores are the softmax over the chosen logits (none of the former apply).
+    `activation` "clipped_swiglu" (with `limit`, `slope`): expert(x) = down(g sigmoid(slope g) (u + 1)), g = min(gate x,
+    limit), u = up x within +- limit. On the device:
     route (one warp per token) -> group the (token, expert) pairs by expert -> one launch for all experts'
     gate/up products with the activation in its epilogue -> one for their down products -> the sum over a
     token's experts with the shared expert in the same kernel. Nothing comes back to the host in between,
@@ -141,7 +147,7 @@ class RoutedExperts(Part):
     params: hidden, experts, top, inter, activation ("silu"), router (tensor name), expert_gate / expert_up /
     expert_down (tensor names with `{}` for the expert's index), shared (a feed-forward PartSpec or None),
     shared_gate (tensor name of a [1, hidden] matrix, or None: the shared expert is added as it is); optional gated,
-    weight_on, correction (tensor name), groups, keep_groups, renormalize, route_scale."""
+    score, limit, slope, weight_on, correction (tensor name), groups, keep_groups, renormalize, route_scale."""
 
     def __init__(self, params, prefix):
         super().__init__(params, prefix)
@@ -155,10 +161,14 @@ class RoutedExperts(Part):
         if self.activation not in ops.EXPERT_ACTIVATIONS:
             raise ValueError(f"routed_experts: unsupported activation {self.activation!r}")
         self.weight_on = p.get("weight_on", "input")
-        if self.weight_on not in ("input", "output") or p.get("score", "sigmoid") != "sigmoid":
-            raise ValueError("routed_experts: built for sigmoid scores that scale the expert's input or its output")
+        self.score = p.get("score", "sigmoid")
+        if self.weight_on not in ("input", "output") or self.score not in ops.ROUTE_SCORES:
+            raise ValueError("routed_experts: built for sigmoid or softmax scores that scale the expert's input or its output")
+        self.limit, self.slope = float(p.get("limit") or 0.0), float(p.get("slope", 1.0))
+        if self.activation == "clipped_swiglu" and not self.limit > 0:
+            raise ValueError("routed_experts: clipped_swiglu needs a positive limit")
         if self.gated and self.activation == "relu2":
-            raise ValueError("routed_experts: gated experts are built with silu or relu")
+            raise ValueError("routed_experts: gated experts are built with silu, relu or the clipped gate")
         if not self.gated and (self.activation != "relu2" or self.weight_on != "output"):
             raise ValueError("routed_experts: experts without a gate are built with the squared relu and weights on their outputs")
         self.renormalize, self.route_scale = bool(p.get("renormalize", False)), float(p.get("route_scale", 1.0))
@@ -168,6 +178,8 @@ class RoutedExperts(Part):
                                 or self.keep_groups * (self.experts // self.groups) < self.top):
             raise ValueError(f"routed_experts: {self.experts} experts in {self.groups} groups of which {self.keep_groups} are kept "
                              f"cannot give a token {self.top} experts")
+        if self.score == "softmax" and (p.get("correction") or self.groups > 1 or self.renormalize or self.route_scale != 1.0):
+            raise ValueError("routed_experts: softmax scores do not combine with corrections, groups, renormalisation or a scale")
         self.correction_name = prefix + p["correction"] if p.get("correction") else None
         self.router_name = prefix + p["router"]
         kinds = ("gate", "up", "down") if self.gated else ("up", "down")
@@ -200,10 +212,12 @@ class RoutedExperts(Part):
         self.router = tensors[self.router_name]
         self.correction = tensors[self.correction_name] if self.correction_name else None
         self._route = dict(correction=self.correction, groups=self.groups, keep_groups=self.keep_groups,
-                           renormalize=self.renormalize, route_scale=self.route_scale)
+                           renormalize=self.renormalize, route_scale=self.route_scale, score=self.score)
+        self._clip = dict(limit=self.limit, slope=self.slope)
         # one copy of the experts' weights serves both forms: where the tensor-core product can fuse the activation
-        # (bfloat16, silu, widths in blocks of 64) every expert's gate and up rows are interleaved for it
-        self.interleaved = (self.gated and runtime.dtype == torch.bfloat16 and self.activation == "silu"
+        # (bfloat16, silu or the clipped gate, widths in blocks of 64) every expert's gate and up rows are interleaved for it
+        self.epilogue = {"silu": "swiglu", "clipped_swiglu": "clipped_swiglu"}.get(self.activation)
+        self.interleaved = (self.gated and runtime.dtype == torch.bfloat16 and self.epilogue is not None
                             and self.inter % ops.SWIGLU_BLOCK == 0)
         stack = ops.interleave_gate_up if self.interleaved else (lambda gate, up: torch.cat((gate, up), dim=0))
         if self.gated:
@@ -265,11 +279,11 @@ class RoutedExperts(Part):
             ops.gemm_tcgen05_grouped(scaled, weights, act, tile_up, self.experts)
             ops.activation(act, act, self.activation)
         elif self.interleaved:
-            ops.gemm_tcgen05_grouped(scaled, weights, act, tile_up, self.experts, epilogue="swiglu")
+            ops.gemm_tcgen05_grouped(scaled, weights, act, tile_up, self.experts, epilogue=self.epilogue, **self._clip)
         else:
             both = torch.empty((rows, 2 * self.inter), dtype=h.dtype, device=h.device)
             ops.gemm_tcgen05_grouped(scaled, weights, both, tile_up, self.experts)
-            ops.gated_act(both, act, self.activation)
+            ops.gated_act(both, act, self.activation, **self._clip)
         y = torch.empty((rows, self.hidden), dtype=h.dtype, device=h.device)     # rounded like every product's output; summed in 32-bit
         ops.gemm_tcgen05_grouped(act, self.down.view(self.experts * self.hidden, self.inter), y, tile_down, self.experts)
         shared = self.shared.forward(h) if self.shared is not None else None
@@ -287,7 +301,7 @@ class RoutedExperts(Part):
         act = torch.empty((pairs, self.inter), dtype=h.dtype, device=h.device)
         on_input = self.weight_on == "input"
         ops.moe_expert_up(h, order, offsets, scores if on_input else None, self.gate_up, act, self.top, self.activation,
-                          self.interleaved, self.gated)
+                          self.interleaved, self.gated, **self._clip)
         y = torch.empty((pairs, self.hidden), dtype=torch.float32, device=h.device)
         ops.moe_expert_down(act, order, offsets, self.down, y)
         shared = self.shared.forward(h) if self.shared is not None else None

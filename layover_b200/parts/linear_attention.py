@@ -252,3 +252,81 @@ class TokenShiftWKV(Part):
         gated = torch.empty((tokens, ch), dtype=h.dtype, device=h.device)
         ops.head_gated_rmsnorm(scanned, proj[:, 3 * ch:], self.norm_w, self.norm_eps, gated, self.heads, self.dim)
         return self.runtime.linear(gated, self.w_o)
+
+
+@register_mixer("gated_linear_attention")
+class GatedLinearAttention(Part):
+    """Linear attention with a decay per key channel that depends on the token. q, k (heads x head_dim) and v (heads x
+    v_head_dim) are plain projections; per head the state S [head_dim, v_head_dim] follows
+
+        alpha_t = sigmoid(W_a2 (W_a1 h) + b)^(1 / tau)                 per head and key channel
+        S <- diag(alpha_t) S + k_t v_t^T,   o_t = head_dim^(-1/2) S^T q_t      (the read-out sees the token's own write)
+
+    Each head's o is RMS-normed over v_head_dim with one weight shared by the heads, multiplied by silu(W_g h) and
+    projected. The state is 32-bit, starts at zero and lives in the request's state slot.
+
+    params: hidden, heads, head_dim, v_head_dim, decay_rank (rows of W_a1), tau, norm_eps, out_scale (default 1: a factor
+    on the heads' outputs, taken into the norm's weight); tensor names q, k, v, gate, a1, a2, a_bias, norm, o relative
+    to the prefix.
+
+    The five projections of h are stacked at load into one product with 32-bit rows; the decays, the recurrence, the
+    norm and the gate are 32-bit arithmetic in a fixed order per token, whatever the cut or the batch."""
+
+    NAMES = ("q", "k", "v", "gate", "a1", "a2", "a_bias", "norm", "o")
+    stackable = True
+
+    def __init__(self, params, prefix):
+        super().__init__(params, prefix)
+        self.require("hidden", "heads", "head_dim", "v_head_dim", "decay_rank", "tau", "norm_eps", *self.NAMES)
+        p = params
+        self.hidden, self.heads, self.dim, self.vdim, self.rank = (
+            int(p[k]) for k in ("hidden", "heads", "head_dim", "v_head_dim", "decay_rank"))
+        if self.dim > 256:
+            raise ValueError(f"gated_linear_attention: head_dim up to 256 is supported, got {self.dim}")
+        self.tau, self.norm_eps, self.out_scale = float(p["tau"]), float(p["norm_eps"]), float(p.get("out_scale", 1.0))
+        if not self.tau > 0:
+            raise ValueError("gated_linear_attention: tau must be positive")
+        self.names = {k: prefix + p[k] for k in self.NAMES}
+        self.qk, self.vv = self.heads * self.dim, self.heads * self.vdim
+        self.w_in = self.w_o = self.a2 = self.a_bias = self.norm_w = None
+
+    def tensor_specs(self):
+        n, hid = self.names, self.hidden
+        return [TensorSpec(n["q"], (self.qk, hid)), TensorSpec(n["k"], (self.qk, hid)), TensorSpec(n["v"], (self.vv, hid)),
+                TensorSpec(n["gate"], (self.vv, hid)), TensorSpec(n["a1"], (self.rank, hid)), TensorSpec(n["a2"], (self.qk, self.rank)),
+                TensorSpec(n["a_bias"], (self.qk,), kind="vector"), TensorSpec(n["norm"], (self.vdim,), kind="vector", init="ones"),
+                TensorSpec(n["o"], (hid, self.vv))]
+
+    def cache_need(self):
+        return StateNeed((self.heads, self.dim, self.vdim), torch.float32)
+
+    def kernel_libraries(self, dtype):
+        return ("wkv", "delta_rule")
+
+    def bind(self, tensors, runtime):
+        super().bind(tensors, runtime)
+        n = self.names
+        rows = [tensors.pop(n[k]) for k in ("q", "k", "v", "gate", "a1")]
+        used = sum(r.shape[0] for r in rows)
+        if used % 16:           # whole 16-byte pieces per output row
+            rows.append(torch.zeros((16 - used % 16, self.hidden), dtype=rows[0].dtype, device=rows[0].device))
+        self.w_in = torch.cat(rows, dim=0).contiguous()                    # [q | k | v | gate | a1 (| padding)]
+        self.a2, self.a_bias, self.w_o = tensors[n["a2"]], tensors[n["a_bias"]], tensors[n["o"]]
+        self.norm_w = tensors[n["norm"]] * self.out_scale
+
+    def mix(self, proj, batch, cache, out) -> None:
+        """From the stacked projection's rows to the gated heads."""
+        tokens, qk, vv = proj.shape[0], self.qk, self.vv
+        gate_at, a_at = 2 * qk + vv, 2 * qk + 2 * vv
+        decay = torch.empty((tokens, qk), dtype=torch.float32, device=proj.device)
+        ops.gate_decay(proj[:, a_at: a_at + self.rank], self.a2, self.a_bias, self.tau, decay)
+        scanned = torch.empty((tokens, vv), dtype=torch.float32, device=proj.device)
+        ops.gated_scan(proj[:, :qk], proj[:, qk: 2 * qk], proj[:, 2 * qk: gate_at], decay, scanned, cache.state, batch,
+                       self.heads, self.dim, self.vdim, self.dim ** -0.5)
+        ops.head_gated_rmsnorm(scanned, proj[:, gate_at: a_at], self.norm_w, self.norm_eps, out, self.heads, self.vdim)
+
+    def forward(self, h: torch.Tensor, batch, cache) -> torch.Tensor:
+        proj = self.runtime.linear(h, self.w_in, out_dtype=torch.float32)
+        gated = torch.empty((h.shape[0], self.vv), dtype=h.dtype, device=h.device)
+        self.mix(proj, batch, cache, gated)
+        return self.runtime.linear(gated, self.w_o)

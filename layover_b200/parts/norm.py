@@ -121,7 +121,8 @@ class RMSNorm(Part):
 class LayerNorm(Part):
     """y = (x - mean) / sqrt(mean((x - mean)^2) + eps) * weight + bias over a 32-bit residual stream.
 
-    params: dim, eps, weight, bias (tensor names relative to the prefix; bias may be None).
+    params: dim, eps, weight, bias (tensor names relative to the prefix; bias may be None), out_scale (default 1: a
+    factor on y, taken into weight and bias when they are bound, in 32-bit).
     `forward(x, delta)` first adds what has not joined the stream yet: `delta` is None, one tensor, or a
     pair of tensors (the two sub-layers of a parallel block, either of which may be None), added as
     x + (a + b) in 32-bit in the same kernel as the norm. The stream must be float32 (a model with
@@ -133,6 +134,7 @@ class LayerNorm(Part):
         self.dim, self.eps = int(params["dim"]), float(params["eps"])
         self.weight_name = prefix + params["weight"]
         self.bias_name = prefix + params["bias"] if params.get("bias") else None
+        self.out_scale = float(params.get("out_scale", 1.0))
         self.weight = self.bias = None
 
     def tensor_specs(self):
@@ -145,6 +147,9 @@ class LayerNorm(Part):
         super().bind(tensors, runtime)
         self.weight = tensors[self.weight_name]
         self.bias = tensors[self.bias_name] if self.bias_name else None
+        if self.out_scale != 1.0:
+            self.weight = self.weight * self.out_scale
+            self.bias = self.bias * self.out_scale if self.bias is not None else None
 
     def kernel_libraries(self, dtype):
         return ("elementwise",)
