@@ -342,7 +342,7 @@ def heads_bias_rope_kv(proj: torch.Tensor, q_out: torch.Tensor, k_pool: torch.Te
     (i < n_freq) instead of i and i + n_freq. `values_from_keys`: the row holds no values; a value head is its key head as
     projected (with the key's bias), before norm and rotation, so vdim = dim. `temperature` = (coef, every): q is also
     multiplied by 1 + coef ln(floor((p + 1) / every) + 1) at position p = positions[t] (int32 [T])."""
-    _need(proj, torch.float32, "proj"); _need(k_pool, q_out.dtype, "k_pool"); _need(v_pool, q_out.dtype, "v_pool")
+    _need_rows(proj, torch.float32, "proj"); _need(k_pool, q_out.dtype, "k_pool"); _need(v_pool, q_out.dtype, "v_pool")
     _need(q_out, None, "q_out"); _need(slot_map, torch.int32, "slot_map")
     tokens = proj.shape[0]
     if values_from_keys and (vdim != dim or v_bias is not None):
