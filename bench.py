@@ -1,7 +1,7 @@
 """Decode and prefill throughput of the engine on one B200, random weights of a named Qwen3 shape.
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--impl ours|reference]
-                    [--config 4b|4b-fp32|8b-mixed|32b-long|topidra|limazen|kirenex|vopozen]
+                    [--config 4b|4b-fp32|8b-mixed|32b-long|topidra|limazen|kirenex|vopozen|fimilix]
 
 A step is one decode step. Every run prints ONE JSON line on standard output.
 
@@ -56,6 +56,12 @@ design the engine has (a recurrence with a decay per token beside latent attenti
 stream itself), at equal width, heads and feed-forward, four layers each: prefill of 2,048 tokens and decode at
 batch 8 for both, then Vopozen's own kernels alone with the like kernel of the other paths beside each.
 
+--config fimilix: the Fimilix design (a parallel block over one LayerNorm of capped attention without a rotation,
+gated linear attention beside it, and routed experts with clipped gates) beside Limazen (the same block and experts
+around attention alone) and Kirenex (a recurrence beside the attention in every layer, dense feed-forward of the
+active width) at equal width and heads, four layers each: prefill of 2,048 tokens and decode at batch 8 for all
+three, then Fimilix's own kernels alone with the like kernels of the other paths (`--only kernels`: those alone).
+
 Peaks come from MEASURED_PEAKS.json beside this file when it exists (else 6.65 TB/s and
 1.59 PFLOP/s, an earlier measurement of the same kind of GPU). Inputs are synthetic token ids;
 weights are seeded random values of the named shape. Weights (8 GB and more) are larger than the
@@ -84,7 +90,8 @@ PROMPT, CONTEXT, PREFILL_TOKENS, PAGE = 2048, 4096, 2048, 16
 FALLBACK_PEAKS = {"hbm_gbs": 6650.0, "bf16_tflops": 1590.0, "bf16_tflops_sustained": 1400.0}
 FP32_TFLOPS = 75.0       # nominal FFMA rate of the part; only the 32-bit path's prefill fraction uses it
 CONFIGS = {"4b": ("qwen3-4b", "bf16"), "4b-fp32": ("qwen3-4b", "fp32"), "8b-mixed": ("qwen3-8b", "bf16"),
-           "32b-long": ("qwen3-32b", "bf16"), "topidra": ("topidra", "bf16"), "limazen": ("limazen", "bf16"), "kirenex": ("kirenex", "bf16"), "vopozen": ("vopozen", "bf16")}
+           "32b-long": ("qwen3-32b", "bf16"), "topidra": ("topidra", "bf16"), "limazen": ("limazen", "bf16"), "kirenex": ("kirenex", "bf16"), "vopozen": ("vopozen", "bf16"),
+           "fimilix": ("fimilix", "bf16")}
 METRIC = "decode tokens/s (Qwen3-4B shape, batch 8, context 2048->4096)"
 
 
@@ -1656,6 +1663,278 @@ def run_vopozen(args, pk, pk_source) -> dict:
             "window_and_chunk": VOPOZEN_SPAN, "sizes": sizes, "kernels": vopozen_kernels(pk)}
 
 
+# --------------------------------------------------------------------------------------- Fimilix beside Limazen and Kirenex
+FIMILIX_SIZES = {   # name: (width, attention and linear heads, KV heads, head size, experts, chosen, expert width)
+    "1024": (1024, 8, 4, 128, 16, 4, 768),
+    "2048": (2048, 16, 8, 128, 32, 4, 1536),
+    "4096": (4096, 32, 8, 128, 32, 4, 3072)}
+FIMILIX_LAYERS, FIMILIX_VOCAB, FIMILIX_RANK, FIMILIX_SPAN, FIMILIX_CAP = 4, 32768, 64, 8192, 30.0
+
+
+def fimilix_trio(size: str):
+    """(Fimilix, Limazen, Kirenex) configurations of equal width, heads, head size and depth. Limazen has the same block
+    and the same experts around attention alone; Kirenex has a recurrence (a gated delta rule of as many heads of the same
+    size) beside the attention in every layer and a dense feed-forward as wide as what a Fimilix token uses. Its window and
+    Limazen's chunk are longer than any request here, so all three attend over every earlier token."""
+    import layover_b200 as lb
+    from layover_b200.config.fimilix import gated_parallel_layer
+    from layover_b200.config.kirenex import parallel_layer
+    from layover_b200.config.limazen import limazen_layer
+
+    width, heads, kv, dim, experts, top, expert_ff = FIMILIX_SIZES[size]
+    layer = gated_parallel_layer(heads, kv, dim, dim, heads, dim, dim, FIMILIX_RANK, softcap=FIMILIX_CAP, q_temp=(0.1, 1024), left_scale=0.7,
+                                 right_scale=0.7, experts=experts, top=top, ff=expert_ff, limit=7.0)
+    fimilix = lb.FimilixConfig(vocab=FIMILIX_VOCAB, width=width, layers=(layer,) * FIMILIX_LAYERS, logit_scale=0.5)
+    chunked = limazen_layer(heads, kv, dim, dim, FIMILIX_SPAN, rot_dims=dim // 2, base=10000.0, factor=2.0, ff=None, experts=experts, top=top,
+                            expert_ff=expert_ff, shared_ff=None)
+    limazen = lb.LimazenConfig(vocab=FIMILIX_VOCAB, width=width, layers=(chunked,) * FIMILIX_LAYERS, logit_softcap=25.0)
+    side = parallel_layer(heads, kv, dim, dim, FIMILIX_SPAN, rot_dims=dim // 2, base=1000000.0, delta_heads=heads, delta_kv_heads=heads,
+                          delta_dim=dim, delta_vdim=dim, taps=KIRENEX_TAPS, ff=top * expert_ff)
+    kirenex = lb.KirenexConfig(vocab=FIMILIX_VOCAB, width=width, layers=(side,) * FIMILIX_LAYERS, max_positions=8192, postln_alpha=1.5)
+    return fimilix, limazen, kirenex
+
+
+def fimilix_kernels(pk: dict) -> dict:
+    """Fimilix's own kernels alone at the 2048 layer size, each with the like kernel of the Limazen, Kirenex, Vopozen or
+    Topidra path: microseconds (kernels back to back in a replayed graph, operands rotating through more memory than the
+    L2 holds) and the fraction of the measured peak that bounds it."""
+    import types
+    import torch
+    from layover_b200 import ops
+
+    width, heads, kv, dim, experts, top, expert_ff = FIMILIX_SIZES["2048"]
+    dev, bf = "cuda", torch.bfloat16
+    hbm, tensor = pk["hbm_gbs"] * 1e9, pk["bf16_tflops"] * 1e12
+    out = {}
+
+    def point(name, fn, calls, nbytes=None, flops=None, peak_flops=None):
+        us = graph_time(fn, calls) * 1000.0
+        row = {"us": round(us, 2)}
+        if nbytes:
+            row["of_hbm"] = round(nbytes / (us * 1e-6) / hbm, 3)
+        if flops:
+            row["of_flops"] = round(flops / (us * 1e-6) / (peak_flops or tensor), 3)
+        out[name] = row
+
+    ROT, page = 6, PAGE
+    n, nkv = heads * dim, kv * dim
+    left_rows, right_rows = n + 2 * nkv, 4 * n + FIMILIX_RANK
+    stacked = left_rows + right_rows
+
+    # ---- the projections of both mixers as one product, and the sum of their outputs as one; beside two products each
+    for tokens in (2048, 8):
+        h = [torch.randn(tokens, width, device=dev, dtype=bf) for _ in range(2)]
+        w = [torch.randn(stacked, width, device=dev, dtype=bf) * 0.02 for _ in range(4)]
+        proj = torch.empty(tokens, stacked, device=dev)
+        point(f"stacked_in_product_{tokens}", lambda i: ops.gemm_bf16(h[i % 2], w[i % 4], proj), 4, flops=2.0 * tokens * stacked * width,
+              nbytes=stacked * width * 2)
+
+        def two_in(i):
+            ops.gemm_bf16(h[i % 2], w[i % 4][:left_rows], proj[:, :left_rows])
+            ops.gemm_bf16(h[i % 2], w[i % 4][left_rows:], proj[:, left_rows:])
+        point(f"like:two_in_products_{tokens}", two_in, 4, flops=2.0 * tokens * stacked * width, nbytes=stacked * width * 2)
+        mixed = [torch.randn(tokens, 2 * n, device=dev, dtype=bf) for _ in range(2)]
+        wo = [torch.randn(width, 2 * n, device=dev, dtype=bf) * 0.02 for _ in range(6)]
+        y = torch.empty(tokens, width, device=dev, dtype=bf)
+        point(f"summed_out_product_{tokens}", lambda i: ops.gemm_bf16(mixed[i % 2], wo[i % 6], y), 6, flops=2.0 * tokens * width * 2 * n,
+              nbytes=width * 2 * n * 2)
+        wo1 = [torch.randn(width, n, device=dev, dtype=bf) * 0.02 for _ in range(12)]
+
+        def two_out(i):
+            ops.gemm_bf16(mixed[i % 2][:, :n], wo1[2 * (i % 6)], y)
+            ops.gemm_bf16(mixed[i % 2][:, n:], wo1[2 * (i % 6) + 1], y)
+        point(f"like:two_out_products_{tokens}", two_out, 6, flops=2.0 * tokens * width * 2 * n, nbytes=width * 2 * n * 2)
+        del h, w, proj, wo, wo1
+        # ---- q/k norm per head, query temperature, page write; beside the same kernel with a rotation
+        pos = torch.arange(tokens, dtype=torch.int32, device=dev)
+        half = torch.empty(tokens, 2, dim // 4, device=dev)
+        ops.rope_table(pos, torch.rand(dim // 4, device=dev), half)
+        slots = torch.arange(tokens, dtype=torch.int32, device=dev)
+        pool = torch.zeros(2, tokens // page + 2, kv, page, dim, device=dev, dtype=bf)
+        qo = torch.empty(tokens, n, device=dev, dtype=bf)
+        wn = torch.ones(dim, device=dev)
+        rows = [torch.randn(tokens, left_rows, device=dev) for _ in range(ROT)]
+        point(f"heads_temperature_kv_{tokens}",
+              lambda i: ops.heads_bias_rope_kv(rows[i % ROT], qo, pool[0], pool[1], None, None, None, None, slots, None, 0, None, heads, kv, dim,
+                                               dim, page, wn, wn, 1e-6, temperature=(0.1, 1024), positions=pos),
+              ROT, nbytes=tokens * left_rows * (4 + 2))
+        point(f"like:heads_rope_kv_{tokens}",
+              lambda i: ops.heads_bias_rope_kv(rows[i % ROT], qo, pool[0], pool[1], None, None, None, half, slots, None, 0, None, heads, kv, dim,
+                                               dim, page, wn, wn, 1e-6), ROT, nbytes=tokens * left_rows * (4 + 2))
+        del rows
+
+    # ---- gated linear attention beside time mixing, the gated delta rule and Topidra's decay scan: a prompt, single tokens
+    prep = ops.delta_prepare_tokens()
+    for tokens, seqs in ((2048, 1), (8, 8), (64, 64)):
+        per = tokens // seqs
+        tag = "prompt2048" if seqs == 1 else f"decode_b{seqs}"
+        floats = heads * dim * dim
+        cu = torch.arange(0, tokens + 1, per, dtype=torch.int32, device=dev)
+        listed = [(s, q0) for s in range(seqs) for q0 in range(0, per, prep)]
+        batch = types.SimpleNamespace(cu_q=cu, state_slots=torch.arange(seqs, dtype=torch.int32, device=dev), n_seqs=seqs, q_lens=[per] * seqs,
+                                      tiles={prep: types.SimpleNamespace(tile_seq=torch.tensor([t[0] for t in listed], dtype=torch.int32, device=dev),
+                                                                         tile_q0=torch.tensor([t[1] for t in listed], dtype=torch.int32, device=dev),
+                                                                         count=len(listed))})
+        lora = [torch.randn(tokens, FIMILIX_RANK, device=dev) for _ in range(ROT)]
+        w2 = torch.randn(n, FIMILIX_RANK, device=dev, dtype=bf) * 0.1
+        w0 = torch.randn(n, device=dev)
+        decay = torch.empty(tokens, n, device=dev)
+        cost = dict(nbytes=tokens * (FIMILIX_RANK + n) * 4 + n * FIMILIX_RANK * 2, flops=2.0 * tokens * n * FIMILIX_RANK, peak_flops=FP32_TFLOPS * 1e12)
+        point(f"gate_decay_{tag}", lambda i: ops.gate_decay(lora[i % ROT], w2, w0, 16.0, decay), ROT, **cost)
+        point(f"like:wkv_decay_{tag}", lambda i: ops.wkv_decay(lora[i % ROT], w2, w0 - 4.0, decay), ROT, **cost)
+        ops.gate_decay(lora[0], w2, w0, 16.0, decay)
+        proj = [torch.randn(tokens, stacked, device=dev) * 0.1 for _ in range(ROT)]
+        at = left_rows
+        state = torch.zeros(ROT, seqs + 1, heads, dim, dim, device=dev)
+        scanned = torch.empty(tokens, n, device=dev)
+        mixed = torch.empty(tokens, 2 * n, device=dev, dtype=bf)
+        point(f"gated_scan_{tag}", lambda i: ops.gated_scan(proj[i % ROT][:, at: at + n], proj[i % ROT][:, at + n: at + 2 * n],
+                                                           proj[i % ROT][:, at + 2 * n: at + 3 * n], decay, scanned, state[i % ROT], batch, heads,
+                                                           dim, dim, dim ** -0.5), ROT,
+              nbytes=tokens * 5 * n * 4 + 2 * seqs * floats * 4, flops=5.0 * tokens * heads * dim * dim, peak_flops=FP32_TFLOPS * 1e12)
+        bonus = torch.rand(heads, dim, device=dev)
+        wstate = state.view(ROT, seqs + 1, floats)
+        point(f"like:wkv_scan_{tag}", lambda i: ops.wkv_scan(proj[i % ROT][:, at: at + n], proj[i % ROT][:, at + n: at + 2 * n],
+                                                            proj[i % ROT][:, at + 2 * n: at + 3 * n], decay, bonus, scanned, wstate[i % ROT], batch,
+                                                            heads, dim), ROT,
+              nbytes=tokens * 5 * n * 4 + 2 * seqs * floats * 4, flops=7.0 * tokens * heads * dim * dim, peak_flops=FP32_TFLOPS * 1e12)
+        wn = torch.ones(dim, device=dev)
+        gated = torch.empty(tokens, n, device=dev, dtype=bf)
+        point(f"head_gated_rmsnorm_wide_rows_{tokens}", lambda i: ops.head_gated_rmsnorm(scanned, proj[i % ROT][:, at + 3 * n: at + 4 * n], wn, 1e-6,
+                                                                                        mixed[:, n:], heads, dim), ROT, nbytes=tokens * n * (4 + 4 + 2))
+        point(f"like:head_gated_rmsnorm_{tokens}", lambda i: ops.head_gated_rmsnorm(scanned, proj[i % ROT][:, at + 3 * n: at + 4 * n], wn, 1e-6, gated,
+                                                                                   heads, dim), ROT, nbytes=tokens * n * (4 + 4 + 2))
+        channels = 3 * n
+        prepared = torch.randn(tokens, channels + 2 * heads, device=dev) * 0.1
+        dstate = torch.zeros(ROT, seqs + 1, floats + 3 * channels, device=dev)
+        point(f"like:delta_scan_{tag}", lambda i: ops.delta_scan(prepared, scanned, dstate[i % ROT], batch, heads, heads, dim, dim), ROT,
+              nbytes=tokens * (channels + n) * 4 + 2 * seqs * floats * 4, flops=6.0 * tokens * heads * dim * dim, peak_flops=FP32_TFLOPS * 1e12)
+        projb = [torch.randn(tokens, 4 * n, device=dev, dtype=bf) for _ in range(ROT)]
+        ldecay = torch.full((heads,), 0.99, device=dev)
+        seg_tokens, segments = ops.scan_segments([per] * seqs, 4 * floats)
+        scratch = torch.empty(segments, heads, dim, dim, device=dev) if segments else None
+        point(f"like:decay_scan_{tag}", lambda i: ops.decay_scan(projb[i % ROT], 0, n, 2 * n, scanned, state[i % ROT], cu, batch.state_slots, ldecay,
+                                                               seqs, heads, dim, dim, "silu", seg_tokens, scratch), ROT,
+              nbytes=tokens * n * (3 * 2 + 4) + 2 * seqs * floats * 4, flops=4.0 * tokens * heads * dim * dim, peak_flops=FP32_TFLOPS * 1e12)
+        del proj, projb, state, dstate, wstate, lora
+
+    # ---- attention with soft-capped scores into wider rows, beside the same kernels without a cap
+    sms = ops.gemm_scratch(torch.device(dev))[2]
+    for tokens, seqs, ctx in ((2048, 1, 2048), (8, 8, 3072), (64, 64, 3072)):
+        pages_per = -(-ctx // page)
+        R = ROT if seqs < 64 else 2
+        table = torch.arange(seqs * pages_per, dtype=torch.int32, device=dev).view(seqs, pages_per)
+        per = tokens // seqs
+        cu = torch.arange(0, tokens + 1, per, dtype=torch.int32, device=dev)
+        lens = torch.full((seqs,), ctx, dtype=torch.int32, device=dev)
+        pools = [torch.randn(2, seqs * pages_per + 1, kv, page, dim, device=dev, dtype=bf) for _ in range(R)]
+        q = torch.randn(tokens, n, device=dev, dtype=bf)
+        o = torch.empty_like(q)
+        wide = torch.empty(tokens, 2 * n, device=dev, dtype=bf)
+        if per > 1:
+            bq = ops.attention_mma_block_queries()
+            tq = torch.arange(0, per, bq, dtype=torch.int32, device=dev)
+            ts = torch.zeros_like(tq)
+            pairs = per * (per + 1) // 2
+            point("capped_attention_prompt2048",
+                  lambda i: ops.attention_prefill_bf16(q, pools[i % R][0], pools[i % R][1], wide[:, :n], table, cu, lens, ts, tq, tq.numel(), heads,
+                                                       kv, dim, page, dim ** -0.5, 0, exact_weights=True, softcap=FIMILIX_CAP, out_scale=0.7), R,
+                  flops=4.0 * heads * dim * 1.25 * pairs)
+            point("like:exact_attention_prompt2048",
+                  lambda i: ops.attention_prefill_bf16(q, pools[i % R][0], pools[i % R][1], o, table, cu, lens, ts, tq, tq.numel(), heads, kv, dim,
+                                                       page, dim ** -0.5, 0, exact_weights=True), R, flops=4.0 * heads * dim * 1.25 * pairs)
+        else:
+            splits, stages = ops.decode_plan(seqs, heads, kv, dim, ctx, sms)
+            point(f"capped_attention_decode_b{seqs}",
+                  lambda i: ops.attention_decode_bf16(q, pools[i % R][0], pools[i % R][1], wide[:, :n], table, cu, lens, None, seqs, heads, kv, dim,
+                                                      page, dim ** -0.5, 0, splits, stages, exact_weights=True, softcap=FIMILIX_CAP, out_scale=0.7),
+                  R, nbytes=seqs * kv * ctx * 2 * dim * 2)
+            point(f"like:exact_attention_decode_b{seqs}",
+                  lambda i: ops.attention_decode_bf16(q, pools[i % R][0], pools[i % R][1], o, table, cu, lens, None, seqs, heads, kv, dim, page,
+                                                      dim ** -0.5, 0, splits, stages, exact_weights=True), R, nbytes=seqs * kv * ctx * 2 * dim * 2)
+        del pools
+        torch.cuda.empty_cache()
+
+    # ---- routed experts: weights by softmax over the chosen, clipped gates; beside Limazen's sigmoid scores and silu
+    clip = dict(limit=7.0, slope=1.702)
+    for tokens in (2048, 8):
+        h = [torch.randn(tokens, width, device=dev, dtype=bf) for _ in range(ROT)]
+        router = torch.randn(experts, width, device=dev) * 0.05
+        ids = torch.empty(tokens, top, dtype=torch.int32, device=dev)
+        scores = torch.empty(tokens, top, device=dev)
+        if tokens > 64:
+            matrix = torch.zeros(-(-experts // 8) * 8, width, device=dev, dtype=bf)
+            matrix[:experts] = router.to(bf)
+            logits = torch.empty(tokens, matrix.shape[0], device=dev)
+
+            def route_product(i, score):
+                ops.gemm_tcgen05(h[i % ROT], matrix, logits)
+                ops.moe_select(logits, experts, top, ids, scores, score=score)
+            point(f"moe_route_product_softmax_{tokens}", lambda i: route_product(i, "softmax"), ROT, nbytes=tokens * width * 2 + experts * width * 2)
+            point(f"like:moe_route_product_{tokens}", lambda i: route_product(i, "sigmoid"), ROT, nbytes=tokens * width * 2 + experts * width * 2)
+        else:
+            point(f"moe_route_softmax_{tokens}", lambda i: ops.moe_route(h[i % ROT], router, top, ids, scores, score="softmax"), ROT,
+                  nbytes=tokens * width * 2 + experts * width * 4)
+            point(f"like:moe_route_{tokens}", lambda i: ops.moe_route(h[i % ROT], router, top, ids, scores), ROT,
+                  nbytes=tokens * width * 2 + experts * width * 4)
+        ops.moe_route(h[0], router, top, ids, scores, score="softmax")
+        pairs = tokens * top
+        gate_up = [torch.randn(experts * 2 * expert_ff, width, device=dev, dtype=bf) * 0.02 for _ in range(2)]
+        if pairs > 4 * experts:
+            rows = ops.moe_padded_rows(pairs, experts)
+            place = torch.empty(pairs, dtype=torch.int32, device=dev)
+            t_up = torch.empty(rows // 128 + 1, dtype=torch.int32, device=dev)
+            t_dn = torch.empty(rows // 128 + 1, dtype=torch.int32, device=dev)
+            ops.moe_group_tiles(ids, experts, place, t_up, t_dn, 2 * expert_ff, width)
+            laid = torch.randn(rows, width, device=dev, dtype=bf)
+            acts = torch.empty(rows, expert_ff, device=dev, dtype=bf)
+            point(f"moe_experts_gate_up_clipped_{tokens}",
+                  lambda i: ops.gemm_tcgen05_grouped(laid, gate_up[i % 2], acts, t_up, experts, "clipped_swiglu", **clip), 2,
+                  flops=2.0 * pairs * 2 * expert_ff * width)
+            point(f"like:moe_experts_gate_up_swiglu_{tokens}", lambda i: ops.gemm_tcgen05_grouped(laid, gate_up[i % 2], acts, t_up, experts, "swiglu"), 2,
+                  flops=2.0 * pairs * 2 * expert_ff * width)
+        else:
+            offsets = torch.empty(experts + 1, dtype=torch.int32, device=dev)
+            order = torch.empty(pairs, dtype=torch.int32, device=dev)
+            ops.moe_group(ids, experts, offsets, order)
+            acts = torch.empty(pairs, expert_ff, device=dev, dtype=bf)
+            used = len(set(ids.flatten().tolist()))       # the experts this step reads
+            stacks = [g.view(experts, 2 * expert_ff, width) for g in gate_up]
+            point(f"moe_experts_gate_up_clipped_{tokens}",
+                  lambda i: ops.moe_expert_up(h[i % ROT], order, offsets, None, stacks[i % 2], acts, top, "clipped_swiglu", True, **clip), 2,
+                  nbytes=used * 2 * expert_ff * width * 2)
+            point(f"like:moe_experts_gate_up_silu_{tokens}",
+                  lambda i: ops.moe_expert_up(h[i % ROT], order, offsets, scores, stacks[i % 2], acts, top, "silu", True), 2,
+                  nbytes=used * 2 * expert_ff * width * 2)
+        del gate_up
+    return out
+
+
+def run_fimilix(args, pk, pk_source) -> dict:
+    import torch
+    import layover_b200 as lb
+
+    gen = torch.Generator().manual_seed(0)
+    sizes = {}
+    for size in FIMILIX_SIZES if args.only != "kernels" else ():
+        row = {}
+        for name, cfg in zip(("fimilix", "limazen", "kirenex"), fimilix_trio(size)):
+            model = lb.random_model(cfg, seed=0, device="cuda", dtype=args.dtype, std=0.02)
+            prefill = prefill_point(model, gen, repeats=5)
+            decode = decode_point(model, args.batch, min(args.steps, 64), args.warmup, gen)
+            row[name] = {"prefill_tok_s": round(prefill["tok_s"], 1), "prefill_ms": round(prefill["ms"], 3),
+                         "decode_tok_s": round(decode["tok_s"], 1), "decode_ms_per_step": round(decode["ms_per_step"], 4),
+                         "launches_per_step": round(decode["launches"] / min(args.steps, 64), 1),
+                         "weight_gb": round(model.weight_bytes() / 1e9, 3)}
+            del model
+            torch.cuda.empty_cache()
+        sizes[size] = row
+    return {"metric": "Fimilix beside Limazen and Kirenex at equal width, heads and active feed-forward width: prefill of 2,048 tokens "
+                      f"and decode at batch {args.batch}, {FIMILIX_LAYERS} layers, vocabulary {FIMILIX_VOCAB}",
+            "dtype": args.dtype, "data": "synthetic token ids, seeded random weights", "peaks": pk_source,
+            "sizes": sizes, "kernels": fimilix_kernels(pk)}
+
+
 def lb_preset(name: str):
     import layover_b200 as lb
     return lb.preset(name)
@@ -1680,6 +1959,8 @@ def run_ours(args) -> dict:
         return run_kirenex(args, pk, pk_source)
     if args.config == "vopozen":
         return run_vopozen(args, pk, pk_source)
+    if args.config == "fimilix":
+        return run_fimilix(args, pk, pk_source)
     if args.only == "kernels":
         return {"only": "kernels", **kernel_points(args.model, pk, with_library=True)}
     if args.only == "plans":
@@ -1826,7 +2107,7 @@ def main(argv=None) -> int:
     parser.add_argument("--config", default="4b", choices=sorted(CONFIGS),
                         help="4b: the headline; 4b-fp32: the 32-bit path; 8b-mixed: 32 mixed requests through the "
                              "scheduler; 32b-long: 8 x 32,768-token contexts; topidra / limazen: that design beside "
-                             "Qwen3 at equal layer sizes, and its kernels alone; kirenex: that design beside Topidra; vopozen: that design beside Kirenex")
+                             "Qwen3 at equal layer sizes, and its kernels alone; kirenex: that design beside Topidra; vopozen: that design beside Kirenex; fimilix: that design beside Limazen and Kirenex")
     parser.add_argument("--model", default=None, help="a preset's name instead of the one --config names")
     parser.add_argument("--dtype", default=None, choices=["bf16", "fp32"])
     parser.add_argument("--batch", type=int, default=8)
