@@ -146,8 +146,18 @@ __device__ __forceinline__ void choose_general(float* z, float* s, float* g, int
   }
 }
 
-// The chosen logits (largest first) become their softmax. One thread.
-__device__ __forceinline__ void softmax_chosen(float* scores, int top) {
+// The chosen logits (largest first) become their softmax. One warp: lane k holds logit k in `mine` where there are at most
+// 32 of them; more are read back from `scores` by lane 0.
+__device__ __forceinline__ void softmax_chosen(float* scores, int top, float mine, int lane) {
+  if (top <= 32) {
+    const float largest = __shfl_sync(0xffffffffu, mine, 0);
+    const float e = lane < top ? expf(mine - largest) : 0.f;
+    const float sum = warp_sum(e);
+    __syncwarp();                                   // lane 0's stores of the logits come first
+    if (lane < top) scores[lane] = e / sum;
+    return;
+  }
+  if (lane != 0) return;
   const float largest = scores[0];
   float sum = 0.f;
   for (int k = 0; k < top; ++k) {
@@ -226,6 +236,7 @@ moe_route_kernel(const T* __restrict__ h, const float* __restrict__ router, cons
       choose_general(z, room, room + experts, experts, top, opt, lane, ids + (size_t)(t0 + t) * top, scores + (size_t)(t0 + t) * top);
       continue;
     }
+    float mine = 0.f;
     for (int k = 0; k < top; ++k) {
       float best = -INFINITY;
       int at = 0x7fffffff;
@@ -240,6 +251,7 @@ moe_route_kernel(const T* __restrict__ h, const float* __restrict__ router, cons
         if (ob > best || (ob == best && oa < at)) { best = ob; at = oa; }
       }
       if (at >= experts) at = k;                    // only when every logit left is NaN or -inf
+      if (lane == k) mine = best;
       if (lane == 0) {
         ids[(size_t)(t0 + t) * top + k] = at;
         scores[(size_t)(t0 + t) * top + k] = opt.softmax ? best : 1.0f / (1.0f + expf(-best));
@@ -247,7 +259,7 @@ moe_route_kernel(const T* __restrict__ h, const float* __restrict__ router, cons
       }
       __syncwarp();
     }
-    if (opt.softmax && lane == 0) softmax_chosen(scores + (size_t)(t0 + t) * top, top);
+    if (opt.softmax) softmax_chosen(scores + (size_t)(t0 + t) * top, top, mine, lane);
   }
 }
 
@@ -274,6 +286,7 @@ moe_select_kernel(const float* __restrict__ logits, long stride, int* __restrict
     choose_general(z, room, room + experts, experts, top, opt, lane, ids + (size_t)t * top, scores + (size_t)t * top);
     return;
   }
+  float mine = 0.f;
   for (int k = 0; k < top; ++k) {
     float best = -INFINITY;
     int at = 0x7fffffff;
@@ -287,6 +300,7 @@ moe_select_kernel(const float* __restrict__ logits, long stride, int* __restrict
       const int oa = __shfl_xor_sync(0xffffffffu, at, o);
       if (ob > best || (ob == best && oa < at)) { best = ob; at = oa; }
     }
+    if (lane == k) mine = best;
     if (at >= experts) at = k;                      // only when every logit left is NaN or -inf
     if (lane == 0) {
       ids[(size_t)t * top + k] = at;
@@ -295,7 +309,7 @@ moe_select_kernel(const float* __restrict__ logits, long stride, int* __restrict
     }
     __syncwarp();
   }
-  if (opt.softmax && lane == 0) softmax_chosen(scores + (size_t)t * top, top);
+  if (opt.softmax) softmax_chosen(scores + (size_t)t * top, top, mine, lane);
 }
 
 // One block: count, scan, place. The order inside a group is the order of arrival; no result depends on it.

@@ -368,7 +368,7 @@ def test_a_layer_norm_with_a_factor_on_its_output(dtype, width):
     close(part.forward(x.cuda(), (a.cuda(), b.cuda())), want, dtype, "all rows")
 
 
-ROUTES = [(16, 5, 64), (7, 3, 40), (5, 1, 24), (2, 2, 16), (1, 1, 16), (64, 8, 128), (130, 6, 72)]       # experts, top, hidden
+ROUTES = [(16, 5, 64), (7, 3, 40), (5, 1, 24), (2, 2, 16), (1, 1, 16), (64, 8, 128), (130, 6, 72), (48, 40, 32)]       # experts, top, hidden
 
 
 def routed_spec(hidden, experts, top, ff, limit):
@@ -398,7 +398,7 @@ def test_the_choice_of_experts_and_their_weights(dtype, tokens, route):
     want_ids, want_w = plain.route(h.to(F), tensors["router"].to(F), top)
     assert factor is None
     firm = firm_rows(h, tensors["router"], top, 1e-4)
-    assert firm.sum() > tokens // 2
+    assert firm.sum() >= tokens // 2
     got_ids, order = ids.cpu().long().sort(dim=1)
     ref_ids, ref_order = want_ids.sort(dim=1)
     assert torch.equal(got_ids[firm], ref_ids[firm])
