@@ -1668,7 +1668,7 @@ FIMILIX_SIZES = {   # name: (width, attention and linear heads, KV heads, head s
     "1024": (1024, 8, 4, 128, 16, 4, 768),
     "2048": (2048, 16, 8, 128, 32, 4, 1536),
     "4096": (4096, 32, 8, 128, 32, 4, 3072)}
-FIMILIX_LAYERS, FIMILIX_VOCAB, FIMILIX_RANK, FIMILIX_SPAN, FIMILIX_CAP = 4, 32768, 64, 8192, 30.0
+FIMILIX_LAYERS, FIMILIX_VOCAB, FIMILIX_RANK, FIMILIX_SPAN, FIMILIX_CAP = 4, 32768, 64, 8192, 25.0
 
 
 def fimilix_trio(size: str):
@@ -1780,9 +1780,9 @@ def fimilix_kernels(pk: dict) -> dict:
         w0 = torch.randn(n, device=dev)
         decay = torch.empty(tokens, n, device=dev)
         cost = dict(nbytes=tokens * (FIMILIX_RANK + n) * 4 + n * FIMILIX_RANK * 2, flops=2.0 * tokens * n * FIMILIX_RANK, peak_flops=FP32_TFLOPS * 1e12)
-        point(f"gate_decay_{tag}", lambda i: ops.gate_decay(lora[i % ROT], w2, w0, 16.0, decay), ROT, **cost)
+        point(f"gate_decay_{tag}", lambda i: ops.gate_decay(lora[i % ROT], w2, w0, 12.0, decay), ROT, **cost)
         point(f"like:wkv_decay_{tag}", lambda i: ops.wkv_decay(lora[i % ROT], w2, w0 - 4.0, decay), ROT, **cost)
-        ops.gate_decay(lora[0], w2, w0, 16.0, decay)
+        ops.gate_decay(lora[0], w2, w0, 12.0, decay)
         proj = [torch.randn(tokens, stacked, device=dev) * 0.1 for _ in range(ROT)]
         at = left_rows
         state = torch.zeros(ROT, seqs + 1, heads, dim, dim, device=dev)

@@ -127,7 +127,7 @@ class FimilixConfig:
         return list(range(self.loop_start)) + span * self.loop_times + list(range(self.loop_stop, len(self.layers)))
 
 
-def gated_parallel_layer(heads, kv_heads, dim, vdim, linear_heads, linear_dim, linear_vdim, decay_rank, tau=16.0, scale=None,
+def gated_parallel_layer(heads, kv_heads, dim, vdim, linear_heads, linear_dim, linear_vdim, decay_rank, tau=12.0, scale=None,
                          softcap=None, q_temp=None, left_scale=1.0, right_scale=1.0, experts=None, top=1, ff=None, limit=7.0) -> dict:
     """One `parallel` entry of `layers`; q_temp = (coef, every)."""
     left = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": scale if scale is not None else dim ** -0.5}

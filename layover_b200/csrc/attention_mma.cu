@@ -759,6 +759,7 @@ void configure_once() {      // once per device: the attribute belongs to the de
   allow_smem(attention_prefill_kernel<256, true, true>, prefill_smem(256));
   allow_smem(attention_prefill_kernel<256, false, true>, prefill_smem(256));
   allow_smem(attention_decode_kernel<128, true, true, false, 3, true>, decode_smem(128));
+  allow_smem(attention_decode_kernel<128, true, false, false, 3, true>, decode_smem(128));
   allow_smem(attention_decode_kernel<128, false, true, false, 3, true>, decode_smem(128));
   allow_smem(attention_decode_kernel<256, true, true, false, 3, true>, decode_smem(256));
   allow_smem(attention_decode_kernel<256, false, true, false, 3, true>, decode_smem(256));
@@ -766,7 +767,9 @@ void configure_once() {      // once per device: the attribute belongs to the de
 
 // the variants with sinks, gates and split weights: three stages, merged through scratch memory
 template <typename... Args>
-int launch_decode_sink(int dim, dim3 grid, size_t smem, cudaStream_t stream, Args... args) {
+int launch_decode_sink(int dim, int group, dim3 grid, size_t smem, cudaStream_t stream, Args... args) {
+  if (dim == 128 && group <= 8)
+    return lb_launch(attention_decode_kernel<128, true, false, false, 3, true>, grid, dim3(THREADS), smem, stream, args...);
   if (dim == 128) return lb_launch(attention_decode_kernel<128, true, true, false, 3, true>, grid, dim3(THREADS), smem, stream, args...);
   if (dim < 128) return lb_launch(attention_decode_kernel<128, false, true, false, 3, true>, grid, dim3(THREADS), smem, stream, args...);
   if (dim == 256) return lb_launch(attention_decode_kernel<256, true, true, false, 3, true>, grid, dim3(THREADS), smem, stream, args...);
@@ -887,7 +890,7 @@ LB_EXPORT int lb_attention_decode_bf16(const void* q, const void* k_pool, const 
   int code;
   const float* no_floats = nullptr;
   if (sink) {
-    code = launch_decode_sink(dim, grid, smem, stream, (const bf16*)q, (const bf16*)k_pool, (const bf16*)v_pool, (bf16*)out,
+    code = launch_decode_sink(dim, q_heads / kv_heads, grid, smem, stream, (const bf16*)q, (const bf16*)k_pool, (const bf16*)v_pool, (bf16*)out,
                               block_table, table_width, cu_q, ctx_len, seq_list, q_heads, kv_heads, dim, page_tokens,
                               scale_log2, window, splits, partials, counters, chunk_shift, page_shift, sinks, gates, keep_first, kv_share, u.cap_in, u.cap_out,
                               out_scale, out_stride);

@@ -56,7 +56,7 @@ CONFIGS = {
     ], loop=(0, 2, 2), logit_scale=3.0),
     # no temperature, no cap, no loop, no scales; every expert chosen
     "plain": config(97, 48, [
-        layer((3, 3, 16, 16, 0.25, None, None), (3, 16, 16, 8, 16.0), (1.0, 1.0), moe(4, 4, 24, 50.0)),
+        layer((3, 3, 16, 16, 0.25, None, None), (3, 16, 16, 8, 12.0), (1.0, 1.0), moe(4, 4, 24, 50.0)),
         layer((2, 1, 32, 16, 0.2, 12.0, None), (2, 160, 16, 4, 5.0), (1.0, 1.0), moe(6, 1, 64, 2.0)),
     ]),
 }
