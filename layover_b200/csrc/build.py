@@ -39,6 +39,7 @@ SOURCES: dict[str, tuple[str, tuple[str, ...]]] = {
     "wkv": ("wkv.cu", ()),
     "latent": ("latent.cu", ()),
     "moe": ("moe.cu", ()),
+    "streams": ("streams.cu", ()),
     "sampling": ("sampling.cu", ()),
     "gemm_tcgen05": ("gemm_tcgen05.cu", ()),
     "attention_mma": ("attention_mma.cu", ()),

@@ -270,10 +270,10 @@ LB_EXPORT int lb_add_rmsnorm(int dtype, void* x, const void* delta, const float*
 }
 
 // ---------------------------------------------------------------- rotary tables
-// table[t][0][i] = cos(pos_t * inv_freq[i]), table[t][1][i] = sin(...), 32-bit (layover/model.py:193-197).
+// table[t][0][i] = amplitude * cos(pos_t * inv_freq[i]), table[t][1][i] = amplitude * sin(...), 32-bit (layover/model.py:193-197).
 // Made once per step and read by every layer, as the reference makes its tables once per call.
 __global__ void rope_table_kernel(const int* __restrict__ positions, const float* __restrict__ inv_freq,
-                                  float* __restrict__ table, int tokens, int n_freq) {
+                                  float* __restrict__ table, int tokens, int n_freq, float amplitude) {
   pdl_launch_dependents();
   pdl_wait();
   const int idx = blockIdx.x * blockDim.x + threadIdx.x;
@@ -281,15 +281,15 @@ __global__ void rope_table_kernel(const int* __restrict__ positions, const float
   const int t = idx / n_freq, i = idx - t * n_freq;
   float sn, cs;
   sincosf((float)positions[t] * inv_freq[i], &sn, &cs);
-  table[((size_t)t * 2) * n_freq + i] = cs;
-  table[((size_t)t * 2 + 1) * n_freq + i] = sn;
+  table[((size_t)t * 2) * n_freq + i] = amplitude * cs;
+  table[((size_t)t * 2 + 1) * n_freq + i] = amplitude * sn;
 }
 
 LB_EXPORT int lb_rope_table(const int* positions, const float* inv_freq, float* table, int tokens, int n_freq,
-                            cudaStream_t stream) {
+                            float amplitude, cudaStream_t stream) {
   const int total = tokens * n_freq;
   if (total <= 0) return 0;
-  lb_launch(rope_table_kernel, (total + 255) / 256, 256, 0, stream, positions, inv_freq, table, tokens, n_freq);
+  lb_launch(rope_table_kernel, (total + 255) / 256, 256, 0, stream, positions, inv_freq, table, tokens, n_freq, amplitude);
   return lb_last_error();
 }
 
@@ -909,6 +909,8 @@ LB_EXPORT int lb_residual_layernorm(int dtype, float* x, const void* delta_a, co
 //   q, k, v += their biases                                              (each null: none)
 //   every q head *= q_norm_w * rsqrt(mean(head^2) + norm_eps), every k head likewise with k_norm_w (weights of
 //   `dim` entries shared by the heads; each null: no norm), before the rotation
+//       (flags & 4: ONE root mean square over all q heads and one over all k heads instead, with a weight per channel
+//       of the whole row)
 //   channels i and i + n_freq of every q and k head (i < n_freq) turn by the token's angle i:
 //       (u, w) -> (u cos - w sin, w cos + u sin), cos/sin from table[t] ([T, 2, n_freq]; null: no rotation)
 //       (flags & 1: neighbouring channels 2i and 2i + 1 turn together instead, by angle i)
@@ -935,6 +937,7 @@ __global__ void heads_bias_rope_kv_kernel(const float* __restrict__ proj, long r
   pdl_launch_dependents();
   pdl_wait();
   const int t = blockIdx.x, nq = q_heads * dim, nk = kv_heads * dim;
+  const bool whole = flags & 4;
   const float* row = proj + (size_t)t * row_stride;
   if (q_norm_w || k_norm_w) {             // a warp per head, lanes over its channels: the same sum for every batch
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
@@ -949,9 +952,20 @@ __global__ void heads_bias_rope_kv_kernel(const float* __restrict__ proj, long r
         ss += v * v;
       }
       ss = warp_sum(ss);
-      if (lane == 0) head_inv[h] = (is_q ? q_norm_w : k_norm_w) ? 1.0f / sqrtf(ss / (float)dim + norm_eps) : 1.f;
+      if (lane == 0) head_inv[h] = whole ? ss : (is_q ? q_norm_w : k_norm_w) ? 1.0f / sqrtf(ss / (float)dim + norm_eps) : 1.f;
     }
     __syncthreads();
+    if (whole) {                          // the heads' sums to one per row: a warp for q, one for k
+      if (warp < 2) {
+        float* sums = head_inv + (warp ? q_heads : 0);
+        const int heads = warp ? kv_heads : q_heads;
+        float ss = 0.f;
+        for (int h = lane; h < heads; h += 32) ss += sums[h];
+        const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)(heads * dim) + norm_eps);
+        for (int h = lane; h < heads; h += 32) sums[h] = inv;
+      }
+      __syncthreads();
+    }
   }
   const float* cs = table ? table + (size_t)t * 2 * n_freq : nullptr;
   const float* sn = cs ? cs + n_freq : nullptr;
@@ -970,6 +984,7 @@ __global__ void heads_bias_rope_kv_kernel(const float* __restrict__ proj, long r
     const float* b = is_q ? q_bias : k_bias;
     if (b) b += h * dim;
     const float* nw = is_q ? q_norm_w : k_norm_w;
+    if (nw && whole) nw += h * dim;
     const float inv = nw ? head_inv[is_q ? h : q_heads + h] : 1.f;
     float v = 0.f;
     if (c < dim) {

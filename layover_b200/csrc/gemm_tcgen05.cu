@@ -84,7 +84,7 @@ template <int BN, typename OutT, int EPI, bool CLUSTER = false>
 __global__ void __launch_bounds__(SMALL_THREADS, SmallTile<BN>::BLOCKS_PER_SM)
 gemm_fewtoken_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_b,
                     OutT* __restrict__ C, long ldc, int rows_a, int rows_b, int K, int splits,
-                    float* __restrict__ partials, unsigned* __restrict__ counters, const HeadsEpilogue he) {
+                    float* __restrict__ partials, unsigned* __restrict__ counters, const HeadsEpilogue he, const LbClip clip) {
   using T = SmallTile<BN>;
   extern __shared__ uint8_t raw_smem[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(raw_smem) + 1023) & ~(uintptr_t)1023);
@@ -312,7 +312,7 @@ gemm_fewtoken_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_con
 #pragma unroll
         for (int i = 0; i < 16; ++i)
           if (c + i < valid_cols) my_partial[(size_t)(c + i) * BM + row] = v[i];
-      } else if (EPI == 1) {
+      } else if (EPI == 1 || EPI == 3) {
         // rows 0..63 of the tile are gate rows, rows 64..127 the up rows of the same features: the
         // upper half hands its values over through shared memory (the ring is drained by now)
         float* handover = reinterpret_cast<float*>(tiles_a);           // [64][17]
@@ -325,7 +325,8 @@ gemm_fewtoken_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_con
 #pragma unroll
           for (int i = 0; i < 16; ++i)
             if (c + i < valid_cols)
-              store_one<OutT>(C + (size_t)(n0 + c + i) * ldc + (m0 >> 1) + row, swiglu_bf16(v[i], handover[row * 17 + i]));
+              store_one<OutT>(C + (size_t)(n0 + c + i) * ldc + (m0 >> 1) + row,
+                              EPI == 3 ? lb_clipped_gate(v[i], handover[row * 17 + i], clip) : swiglu_bf16(v[i], handover[row * 17 + i]));
         }
         __syncthreads();
       } else {
@@ -1017,7 +1018,7 @@ static inline bool lb_gemm_pair_enabled() {
 
 template <typename OutT, int EPI = 0>
 int launch_pair(const CUtensorMap& map_a, const CUtensorMap& map_b, void* C, long ldc, const Problem& pb, bool vector_ok,
-                cudaStream_t stream, const HeadsEpilogue& he = HeadsEpilogue{}) {
+                cudaStream_t stream, const HeadsEpilogue& he = HeadsEpilogue{}, LbClip clip = LbClip{}) {
   constexpr int BN = 256;
   using T = Tile<BN, false, true>;
   auto kernel = gemm_tcgen05_kernel<BN, false, OutT, EPI, true>;
@@ -1076,13 +1077,13 @@ int launch_pair(const CUtensorMap& map_a, const CUtensorMap& map_b, void* C, lon
   float* partials = sch.last_splits > 1 ? pb.scratch : nullptr;
   const int code = lb_launch_cluster_dims(kernel, dim3(2 * pairs), dim3(persistent_threads(EPI)), (size_t)T::SMEM, stream,
                                           dim3(2, 1, 1), map_a, map_b, (OutT*)C, ldc, pb.rows_a, pb.rows_b, sch, partials,
-                                          pb.counters, vector_ok, he, (const int*)nullptr, LbClip{});
+                                          pb.counters, vector_ok, he, (const int*)nullptr, clip);
   return code ? code : lb_last_error();
 }
 
 template <int BN, typename OutT, int EPI = 0>
 int launch_fewtoken(const CUtensorMap& map_a, const CUtensorMap& map_b, void* C, long ldc, const Problem& pb,
-                    cudaStream_t stream) {
+                    cudaStream_t stream, LbClip clip = LbClip{}) {
   using T = SmallTile<BN>;
   auto kernel = gemm_fewtoken_kernel<BN, OutT, EPI>;
   static LbPerDeviceOnce configured;
@@ -1119,13 +1120,13 @@ int launch_fewtoken(const CUtensorMap& map_a, const CUtensorMap& map_b, void* C,
       }
       const int code = lb_launch_cluster(cluster_kernel, grid, dim3(SMALL_THREADS), (size_t)T::SMEM_CLUSTER, stream,
                                          (unsigned)splits, map_a, map_b, (OutT*)C, ldc, pb.rows_a, pb.rows_b, pb.K,
-                                         splits, (float*)nullptr, (unsigned*)nullptr, HeadsEpilogue{});
+                                         splits, (float*)nullptr, (unsigned*)nullptr, HeadsEpilogue{}, LbClip{});
       return code ? code : lb_last_error();
     }
   }
   const int code = lb_launch(kernel, grid, dim3(SMALL_THREADS), (size_t)T::SMEM, stream, map_a, map_b, (OutT*)C, ldc,
                              pb.rows_a, pb.rows_b, pb.K, splits, splits > 1 ? pb.scratch : (float*)nullptr, pb.counters,
-                             HeadsEpilogue{});
+                             HeadsEpilogue{}, clip);
   return code ? code : lb_last_error();
 }
 
@@ -1150,7 +1151,7 @@ int launch_heads(const CUtensorMap& map_a, const CUtensorMap& map_b, const Probl
   dim3 grid(tiles, 1, splits);
   const int code = lb_launch_cluster(kernel, grid, dim3(SMALL_THREADS), (size_t)T::SMEM_CLUSTER, stream, (unsigned)splits,
                                      map_a, map_b, (bf16*)nullptr, 0L, pb.rows_a, pb.rows_b, pb.K, splits, (float*)nullptr,
-                                     (unsigned*)nullptr, he);
+                                     (unsigned*)nullptr, he, LbClip{});
   return code ? code : lb_last_error();
 }
 }  // namespace
@@ -1186,13 +1187,17 @@ LB_EXPORT int lb_gemm_tcgen05_supports(const void* A, const void* W, int K, long
 // C[M, N] = A[M, K] W[N, K]^T. out_dtype: LB_BF16 or LB_F32. `scratch` (floats) and `counters`
 // (zeroed once by the caller, `n_counters` of them) serve the split-K path; without them K is
 // never split. `sm_count` sizes the grid; `max_splits` > 0 caps the splitting. `epilogue` 1: W's rows
-// come as blocks of 64 gate rows + 64 up rows and C[M, N / 2] = silu(gate) * up (bfloat16 only).
+// come as blocks of 64 gate rows + 64 up rows and C[M, N / 2] = silu(gate) * up (bfloat16 only). 3: the same row blocks
+// with the clipped gate of `limit` and `slope`, for at most 16 tokens and for more than 128.
 LB_EXPORT int lb_gemm_tcgen05(const void* A, const void* W, void* C, int out_dtype, int M, int N, int K, long lda,
                               long ldw, long ldc, float* scratch, long scratch_floats, unsigned* counters,
-                              int n_counters, int sm_count, int max_splits, int epilogue, cudaStream_t stream) {
+                              int n_counters, int sm_count, int max_splits, int epilogue, float limit, float slope,
+                              cudaStream_t stream) {
   if (M <= 0 || N <= 0) return 0;
-  if (epilogue != 0 && epilogue != 1) return LB_ERR_SIZE;
-  if (epilogue == 1 && (N % 128 != 0 || out_dtype != LB_BF16)) return LB_ERR_SIZE;   // blocks of 64 gate + 64 up rows
+  if (epilogue != 0 && epilogue != 1 && epilogue != 3) return LB_ERR_SIZE;
+  if (epilogue == 3 && M > 16 && M <= 128) return LB_ERR_SIZE;
+  if (epilogue && (N % 128 != 0 || out_dtype != LB_BF16)) return LB_ERR_SIZE;   // blocks of 64 gate + 64 up rows
+  const LbClip clip{limit, slope};
   if (!lb_gemm_tcgen05_supports(A, W, K, lda, ldw)) return LB_ERR_ALIGN;
   if (out_dtype != LB_BF16 && out_dtype != LB_F32) return LB_ERR_DTYPE;
   if (sm_count < 1) sm_count = 1;
@@ -1219,6 +1224,7 @@ LB_EXPORT int lb_gemm_tcgen05(const void* A, const void* W, void* C, int out_dty
     if (make_map(&map_half, W, N, K, ldw, 128)) {
       int code;
       if (epilogue == 1) code = launch_pair<bf16, 1>(map_a, map_half, C, ldc, pb, vector_ok, stream);
+      else if (epilogue == 3) code = launch_pair<bf16, 3>(map_a, map_half, C, ldc, pb, vector_ok, stream, HeadsEpilogue{}, clip);
       else if (out_dtype == LB_BF16) code = launch_pair<bf16>(map_a, map_half, C, ldc, pb, vector_ok, stream);
       else code = launch_pair<float>(map_a, map_half, C, ldc, pb, vector_ok, stream);
       if (code != -1) return code;
@@ -1243,6 +1249,11 @@ LB_EXPORT int lb_gemm_tcgen05(const void* A, const void* W, void* C, int out_dty
     }
     if (bn == 128) return launch<128, false, bf16, 1>(map_a, map_b, C, ldc, pb, vector_ok, stream);
     return launch<256, false, bf16, 1>(map_a, map_b, C, ldc, pb, vector_ok, stream);
+  }
+  if (epilogue == 3) {
+    if (swap) return launch_fewtoken<16, bf16, 3>(map_a, map_b, C, ldc, pb, stream, clip);
+    if (bn == 128) return launch<128, false, bf16, 3>(map_a, map_b, C, ldc, pb, vector_ok, stream, nullptr, clip);
+    return launch<256, false, bf16, 3>(map_a, map_b, C, ldc, pb, vector_ok, stream, nullptr, clip);
   }
   // 32..128 tokens and a weight with fewer 128-row tiles than SMs: the persistent kernel, whose
   // blocks add up the partial tiles together, takes 8 splits well (measured: 11 us against 18 us

@@ -12,31 +12,31 @@
 #include "common.cuh"
 
 namespace {
-// One block per token over its 32-bit projection row. With `dkv_off` >= 0 the row holds [latent: rank |
-// rotated key part: rot] there: c = latent * rsqrt(mean(latent^2) + eps) * norm_w goes to channels [0, rank) of
-// the token's cache row, the rotated key part to [rank, rank + rot), zeros up to `room`. q at `q_off` is
-// q_heads x [dim | rot]: the rotated part of every head goes to channels [rank, rank + rot) of q_out's head (zeros
-// up to room); channels [0, rank) are left to the product that folds the key map into the query.
-// Rotation: channels 2i and 2i + 1 turn by the token's angle i, (u, v) -> (u cos - v sin, v cos + u sin), cos/sin
-// from table[t] ([T, 2, rot / 2]).
+// The rotated parts: channels 2i and 2i + 1 turn by the token's angle i, (u, v) -> (u cos - v sin, v cos + u sin), cos/sin
+// from the token's row of the step's table [T, 2, rot / 2]. Channel c of `part`, turned:
+template <typename TA>
+__device__ __forceinline__ float turned_channel(const TA* part, const float* cs, int half, int c) {
+  const int i = c >> 1;
+  const float u = Elem<TA>::load(part + 2 * i), v = Elem<TA>::load(part + 2 * i + 1), co = cs[i], si = cs[half + i];
+  return (c & 1) ? v * co + u * si : u * co - v * si;
+}
+
+// One block per token over its 32-bit projection row. The row holds [latent: rank | rotated key part: rot] at `dkv_off`:
+// c = latent * rsqrt(mean(latent^2) + eps) * norm_w goes to channels [0, rank) of the token's cache row, the rotated key
+// part to [rank, rank + rot), zeros up to `room`. With `cq_rank` > 0 the row also holds the latent of the queries at
+// `cq_off`; it is normed likewise with `cq_norm_w` and left in cq_out [T, cq_rank] for the product that follows.
 template <typename T>
-__global__ void latent_rows_kernel(const float* __restrict__ proj, long row_stride, int q_off, int dkv_off,
-                                   const float* __restrict__ norm_w, float eps, const float* __restrict__ table,
-                                   const int* __restrict__ slot_map, T* __restrict__ k_pool, T* __restrict__ q_out,
-                                   int q_heads, int dim, int rot, int rank, int room, int page_tokens) {
+__global__ void latent_rows_kernel(const float* __restrict__ proj, long row_stride, int dkv_off, const float* __restrict__ norm_w,
+                                   float eps, const float* __restrict__ table, const int* __restrict__ slot_map,
+                                   T* __restrict__ k_pool, int rot, int rank, int room, int page_tokens, int cq_off, int cq_rank,
+                                   const float* __restrict__ cq_norm_w, T* __restrict__ cq_out) {
   __shared__ float scratch[33];
   pdl_launch_dependents();
   pdl_wait();
   const int t = blockIdx.x, half = rot >> 1;
   const float* row = proj + (size_t)t * row_stride;
-  const float* cs = table + (size_t)t * 2 * half;
-  const float* sn = cs + half;
-  auto turned = [&](const float* part, int c) {      // channel c of a rotated part
-    const int i = c >> 1;
-    const float u = part[2 * i], v = part[2 * i + 1];
-    return (c & 1) ? v * cs[i] + u * sn[i] : u * cs[i] - v * sn[i];
-  };
   if (dkv_off >= 0) {
+    const float* cs = table + (size_t)t * 2 * half;
     const float* latent = row + dkv_off;
     float ss = 0.f;
     for (int c = threadIdx.x; c < rank; c += blockDim.x) ss += latent[c] * latent[c];
@@ -46,29 +46,37 @@ __global__ void latent_rows_kernel(const float* __restrict__ proj, long row_stri
     for (int c = threadIdx.x; c < room; c += blockDim.x) {
       float v = 0.f;
       if (c < rank) v = latent[c] * inv * norm_w[c];
-      else if (c < rank + rot) v = turned(latent + rank, c - rank);
+      else if (c < rank + rot) v = turned_channel(latent + rank, cs, half, c - rank);
       Elem<T>::store(dst + c, v);
     }
   }
-  const int tail = room - rank;
-  for (int i = threadIdx.x; i < q_heads * tail; i += blockDim.x) {
-    const int h = i / tail, c = i - h * tail;
-    const float v = c < rot ? turned(row + q_off + h * (dim + rot) + dim, c) : 0.f;
-    Elem<T>::store(q_out + ((size_t)t * q_heads + h) * room + rank + c, v);
+  if (cq_rank > 0) {
+    const float* latent = row + cq_off;
+    float ss = 0.f;
+    for (int c = threadIdx.x; c < cq_rank; c += blockDim.x) ss += latent[c] * latent[c];
+    const float inv = 1.0f / sqrtf(block_sum(ss, scratch) / (float)cq_rank + eps);
+    for (int c = threadIdx.x; c < cq_rank; c += blockDim.x) Elem<T>::store(cq_out + (size_t)t * cq_rank + c, latent[c] * inv * cq_norm_w[c]);
   }
 }
 
-// out[t, h, n] = sum_k a[t, h, k] * w[h, n, k]  (* sigmoid(gate[t, h * N + n])), one product per head:
+// out[t, h, n] = sum_k a[t, h, k] * w[h, n, k]  (* sigmoid(gate[t, h * gate_head + n * gate_n])), one product per head:
+// a gate per channel (gate_head = N, gate_n = 1) or per head (1, 0);
 // a rows `a_row` elements apart with heads `a_head` apart, out likewise, w [heads, N, K] dense. 32-bit sums in
-// the order of k, so a row's result does not depend on the batch or on the tile. A block: 8 TPT tokens x 64 outputs of
+// the order of k, so a row's result does not depend on the batch or on the tile. With `tail.room` > 0 a head of `a` has `rot`
+// more channels behind its K: they are turned by the token's angles and follow the N outputs, zeros up to `room` channels
+// (what makes a query whole: its folded part and its rotated part). A block: 8 TPT tokens x 64 outputs of
 // one head, TPT tokens x 4 outputs a thread (2 for a few tokens, 8 for many: 32 products for 12 reads of shared memory).
 constexpr int HL_OUT = 64, HL_K = 32;
+struct RotatedTail {
+  const float* table;     // [T, 2, rot / 2]
+  int rot, room;
+};
 
 template <typename TA, typename T, int TPT>
 __global__ void __launch_bounds__(128)
 heads_linear_kernel(const TA* __restrict__ a, long a_row, long a_head, const T* __restrict__ w, T* __restrict__ out,
-                    long out_row, long out_head, const float* __restrict__ gate, long gate_row, int tokens, int n_out,
-                    int k_dim) {
+                    long out_row, long out_head, const float* __restrict__ gate, long gate_row, int gate_head, int gate_n,
+                    int tokens, int n_out, int k_dim, const RotatedTail tail) {
   constexpr int HL_TOKENS = 8 * TPT;
   __shared__ float a_s[HL_TOKENS][HL_K + 1];
   __shared__ float w_s[HL_OUT][HL_K + 1];
@@ -112,42 +120,55 @@ heads_linear_kernel(const TA* __restrict__ a, long a_row, long a_head, const T* 
       const int n = n0 + tx + 16 * j;
       if (n >= n_out) continue;
       float v = acc[r][j];
-      if (gate) v *= 1.0f / (1.0f + expf(-gate[(size_t)t * gate_row + (size_t)h * n_out + n]));
+      if (gate) v *= 1.0f / (1.0f + expf(-gate[(size_t)t * gate_row + (size_t)h * gate_head + (size_t)n * gate_n]));
       Elem<T>::store(out + (size_t)t * out_row + (size_t)h * out_head + n, v);
+    }
+  }
+  if (tail.room > 0 && blockIdx.y == 0) {
+    for (int i = threadIdx.x; i < HL_TOKENS * tail.room; i += 128) {
+      const int r = i / tail.room, c = i - r * tail.room, t = t0 + r;
+      if (t >= tokens) break;
+      float v = 0.f;
+      if (c < tail.rot)
+        v = turned_channel(a + (size_t)t * a_row + (size_t)h * a_head + k_dim, tail.table + (size_t)t * tail.rot, tail.rot >> 1, c);
+      Elem<T>::store(out + (size_t)t * out_row + (size_t)h * out_head + n_out + c, v);
     }
   }
 }
 }  // namespace
 
-LB_EXPORT int lb_latent_rows(int dtype, const float* proj, long row_stride, int q_off, int dkv_off, const float* norm_w,
-                             float eps, const float* table, const int* slot_map, void* k_pool, void* q_out, int tokens,
-                             int q_heads, int dim, int rot, int rank, int room, int page_tokens, cudaStream_t stream) {
+LB_EXPORT int lb_latent_rows(int dtype, const float* proj, long row_stride, int dkv_off, const float* norm_w, float eps,
+                             const float* table, const int* slot_map, void* k_pool, int tokens, int rot, int rank, int room,
+                             int page_tokens, int cq_off, int cq_rank, const float* cq_norm_w, void* cq_out, cudaStream_t stream) {
   if (tokens <= 0) return 0;
-  if (q_heads <= 0 || dim <= 0 || rot < 0 || rot % 2 || rank <= 0 || room < rank + rot || page_tokens <= 0 || !table ||
-      (dkv_off >= 0 && (!norm_w || !slot_map || !k_pool)))
+  if (rot < 0 || rot % 2 || cq_rank < 0 || (cq_rank > 0 && (cq_off < 0 || !cq_norm_w || !cq_out)) || (dkv_off < 0 && cq_rank == 0) ||
+      (dkv_off >= 0 && (rank <= 0 || room < rank + rot || page_tokens <= 0 || !table || !norm_w || !slot_map || !k_pool)))
     return LB_ERR_SIZE;
   if (dtype == LB_F32)
-    lb_launch(latent_rows_kernel<float>, tokens, 128, 0, stream, proj, row_stride, q_off, dkv_off, norm_w, eps, table, slot_map,
-              (float*)k_pool, (float*)q_out, q_heads, dim, rot, rank, room, page_tokens);
+    lb_launch(latent_rows_kernel<float>, tokens, 128, 0, stream, proj, row_stride, dkv_off, norm_w, eps, table, slot_map,
+              (float*)k_pool, rot, rank, room, page_tokens, cq_off, cq_rank, cq_norm_w, (float*)cq_out);
   else if (dtype == LB_BF16)
-    lb_launch(latent_rows_kernel<bf16>, tokens, 128, 0, stream, proj, row_stride, q_off, dkv_off, norm_w, eps, table, slot_map,
-              (bf16*)k_pool, (bf16*)q_out, q_heads, dim, rot, rank, room, page_tokens);
+    lb_launch(latent_rows_kernel<bf16>, tokens, 128, 0, stream, proj, row_stride, dkv_off, norm_w, eps, table, slot_map,
+              (bf16*)k_pool, rot, rank, room, page_tokens, cq_off, cq_rank, cq_norm_w, (bf16*)cq_out);
   else
     return LB_ERR_DTYPE;
   return lb_last_error();
 }
 
-// a_float: a is 32-bit whatever `dtype` (the projection's unrounded rows); w and out are of `dtype`.
+// a_float: a is 32-bit whatever `dtype` (the projection's unrounded rows); w and out are of `dtype`. table null: no tail.
 LB_EXPORT int lb_heads_linear(int dtype, int a_float, const void* a, long a_row, long a_head, const void* w, void* out,
-                              long out_row, long out_head, const float* gate, long gate_row, int tokens, int heads, int n_out,
-                              int k_dim, cudaStream_t stream) {
+                              long out_row, long out_head, const float* gate, long gate_row, int gate_per_head, int tokens, int heads,
+                              int n_out, int k_dim, const float* table, int rot, int tail_room, cudaStream_t stream) {
   if (tokens <= 0) return 0;
-  if (heads <= 0 || heads > 65535 || n_out <= 0 || k_dim <= 0 || (n_out + HL_OUT - 1) / HL_OUT > 65535) return LB_ERR_SIZE;
-  const int tpt = tokens >= 256 ? 8 : 2;
+  if (heads <= 0 || heads > 65535 || n_out <= 0 || k_dim <= 0 || (n_out + HL_OUT - 1) / HL_OUT > 65535 ||
+      (table && (rot < 0 || rot % 2 || tail_room < rot)))
+    return LB_ERR_SIZE;
+  const RotatedTail tail{table, table ? rot : 0, table ? tail_room : 0};
+  const int tpt = tokens >= 256 ? 8 : 2, gate_head = gate_per_head ? 1 : n_out, gate_n = gate_per_head ? 0 : 1;
   dim3 grid((tokens + 8 * tpt - 1) / (8 * tpt), (n_out + HL_OUT - 1) / HL_OUT, heads);
 #define LB_HL_T(TA, T, TPT)                                                                                                    \
   lb_launch(heads_linear_kernel<TA, T, TPT>, grid, 128, 0, stream, (const TA*)a, a_row, a_head, (const T*)w, (T*)out, out_row, \
-            out_head, gate, gate_row, tokens, n_out, k_dim)
+            out_head, gate, gate_row, gate_head, gate_n, tokens, n_out, k_dim, tail)
 #define LB_HL(TA, T)             \
   do {                           \
     if (tpt == 8) LB_HL_T(TA, T, 8); \

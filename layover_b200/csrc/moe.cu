@@ -6,7 +6,7 @@
 //   route     z = W_router h in 32-bit, one warp per token; score = sigmoid(z); the `top` largest z
 //             (ties: the lower index) with their scores; optionally one more 32-bit dot product per
 //             token, sigmoid(w_shared . h), the factor of a shared expert; or the scores are the softmax over
-//             the chosen logits alone
+//             the chosen logits alone, or over all of them
 //   group     offsets[e] .. offsets[e + 1] = the places of expert e's pairs in `order`, order[place] =
 //             pair = token * top + k
 //   products  for every expert e and every pair in its group
@@ -61,26 +61,36 @@ template <> struct Piece<bf16> {
 // How a token's experts are chosen beyond "the `top` largest logits", for routers that need it:
 //   correction  float [experts] or null: the choice is made on sigmoid(z) + correction, the weights are sigmoid(z)
 //   groups      > 1: the experts are `groups` equal groups of neighbours; a group's score is the sum of its two largest
-//               choice scores (its only one, if a group has one expert); only experts of the `keep` best groups can be
-//               chosen (ties: the lower index)
+//               choice scores (its only one, if a group has one expert), or, with `group_best`, its largest one; only
+//               experts of the `keep` best groups can be chosen (ties: the lower index)
 //   renorm      the chosen weights are divided by their sum (+ 1e-20)
 //   scale       then multiplied by this
-//   softmax     the choice is made on the logits and the weights are the softmax over the chosen logits; with none of
-//               the others
+//   softmax     ROUTE_CHOSEN: the choice is made on the logits and the weights are the softmax over the chosen logits;
+//               with none of the others. ROUTE_ALL: a score is the softmax over all experts instead of sigmoid(z)
 // All of it is one warp's work per token on 32-bit numbers in shared memory.
+enum RouteScore { ROUTE_SIGMOID = 0, ROUTE_CHOSEN = 1, ROUTE_ALL = 2 };
 struct RouteOptions {
   const float* correction;
-  int groups, keep, renorm;
+  int groups, keep, group_best, renorm;
   float scale;
   int softmax;
-  __host__ __device__ bool general() const { return correction || groups > 1 || renorm || scale != 1.f; }
+  __host__ __device__ bool general() const { return correction || groups > 1 || renorm || scale != 1.f || softmax == ROUTE_ALL; }
 };
 
 // z [experts]: the token's logits (overwritten); s [experts] and g [groups]: room for the scores. One warp.
 __device__ __forceinline__ void choose_general(float* z, float* s, float* g, int experts, int top, const RouteOptions& opt,
                                                int lane, int* ids, float* scores) {
+  float largest = 0.f, total = 1.f;
+  if (opt.softmax == ROUTE_ALL) {
+    largest = -INFINITY;
+    for (int e = lane; e < experts; e += 32) largest = fmaxf(largest, z[e]);
+    largest = warp_max(largest);
+    total = 0.f;
+    for (int e = lane; e < experts; e += 32) total += expf(z[e] - largest);
+    total = warp_sum(total);
+  }
   for (int e = lane; e < experts; e += 32) {
-    const float score = 1.0f / (1.0f + expf(-z[e]));
+    const float score = opt.softmax == ROUTE_ALL ? expf(z[e] - largest) / total : 1.0f / (1.0f + expf(-z[e]));
     s[e] = score;
     z[e] = score + (opt.correction ? opt.correction[e] : 0.f);
   }
@@ -93,7 +103,7 @@ __device__ __forceinline__ void choose_general(float* z, float* s, float* g, int
         const float v = z[e];
         if (v > m1) { m2 = m1; m1 = v; } else if (v > m2) { m2 = v; }
       }
-      g[i] = size >= 2 ? m1 + m2 : m1;
+      g[i] = size >= 2 && !opt.group_best ? m1 + m2 : m1;
     }
     __syncwarp();
     for (int k = 0; k < opt.keep; ++k) {          // a kept group is marked with a NaN, which no comparison picks again
@@ -254,12 +264,12 @@ moe_route_kernel(const T* __restrict__ h, const float* __restrict__ router, cons
       if (lane == k) mine = best;
       if (lane == 0) {
         ids[(size_t)(t0 + t) * top + k] = at;
-        scores[(size_t)(t0 + t) * top + k] = opt.softmax ? best : 1.0f / (1.0f + expf(-best));
+        scores[(size_t)(t0 + t) * top + k] = opt.softmax == ROUTE_CHOSEN ? best : 1.0f / (1.0f + expf(-best));
         z[at] = -INFINITY;                          // taken
       }
       __syncwarp();
     }
-    if (opt.softmax) softmax_chosen(scores + (size_t)(t0 + t) * top, top, mine, lane);
+    if (opt.softmax == ROUTE_CHOSEN) softmax_chosen(scores + (size_t)(t0 + t) * top, top, mine, lane);
   }
 }
 
@@ -304,12 +314,12 @@ moe_select_kernel(const float* __restrict__ logits, long stride, int* __restrict
     if (at >= experts) at = k;                      // only when every logit left is NaN or -inf
     if (lane == 0) {
       ids[(size_t)t * top + k] = at;
-      scores[(size_t)t * top + k] = opt.softmax ? best : 1.0f / (1.0f + expf(-best));
+      scores[(size_t)t * top + k] = opt.softmax == ROUTE_CHOSEN ? best : 1.0f / (1.0f + expf(-best));
       z[at] = -INFINITY;                            // taken
     }
     __syncwarp();
   }
-  if (opt.softmax) softmax_chosen(scores + (size_t)t * top, top, mine, lane);
+  if (opt.softmax == ROUTE_CHOSEN) softmax_chosen(scores + (size_t)t * top, top, mine, lane);
 }
 
 // One block: count, scan, place. The order inside a group is the order of arrival; no result depends on it.
@@ -699,21 +709,22 @@ static void launch_route(const void* h, const float* router, const float* shared
 #undef LB_ROUTE_ARGS
 }
 
-static bool route_options(RouteOptions& opt, const float* correction, int groups, int keep, int renorm, float scale, int softmax,
-                          int experts) {
-  opt = RouteOptions{correction, groups > 1 ? groups : 0, keep, renorm, scale, softmax};
-  if (softmax && opt.general()) return false;
+static bool route_options(RouteOptions& opt, const float* correction, int groups, int keep, int group_best, int renorm, float scale,
+                          int softmax, int experts) {
+  opt = RouteOptions{correction, groups > 1 ? groups : 0, keep, group_best, renorm, scale, softmax};
+  if (softmax < ROUTE_SIGMOID || softmax > ROUTE_ALL || (softmax == ROUTE_CHOSEN && opt.general())) return false;
   return !(groups > 1 && (experts % groups || keep <= 0 || keep > groups)) && scale > 0.f;
 }
 
-// correction, groups, keep, renorm, scale, softmax: see RouteOptions (null, 0, 0, 0, 1, 0: the `top` largest logits and their sigmoids).
+// correction, groups, keep, group_best, renorm, scale, softmax: see RouteOptions (null, 0, 0, 0, 0, 1, 0: the `top` largest logits and their sigmoids).
 LB_EXPORT int lb_moe_route(int dtype, const void* h, const float* router, const float* shared_w, int* ids, float* scores,
                            float* shared_factor, int tokens, int hidden, int experts, int top, const float* correction,
-                           int groups, int keep, int renorm, float scale, int softmax, cudaStream_t stream) {
+                           int groups, int keep, int group_best, int renorm, float scale, int softmax,
+                           cudaStream_t stream) {
   if (tokens <= 0) return 0;
   RouteOptions opt;
   if (hidden <= 0 || experts <= 0 || top <= 0 || top > experts || experts > 1024 || (shared_w && !shared_factor) ||
-      !route_options(opt, correction, groups, keep, renorm, scale, softmax, experts))
+      !route_options(opt, correction, groups, keep, group_best, renorm, scale, softmax, experts))
     return LB_ERR_SIZE;
   if (dtype == LB_F32) launch_route<float>(h, router, shared_w, ids, scores, shared_factor, tokens, hidden, experts, top, opt, stream);
   else if (dtype == LB_BF16) launch_route<bf16>(h, router, shared_w, ids, scores, shared_factor, tokens, hidden, experts, top, opt, stream);
@@ -724,12 +735,12 @@ LB_EXPORT int lb_moe_route(int dtype, const void* h, const float* router, const 
 // ids, scores (and shared_factor, from column `experts`, when not null) from logits [tokens, >= experts (+ 1)] with row
 // stride `stride` floats.
 LB_EXPORT int lb_moe_select(const float* logits, long stride, int* ids, float* scores, float* shared_factor, int tokens,
-                            int experts, int top, const float* correction, int groups, int keep, int renorm, float scale,
-                            int softmax, cudaStream_t stream) {
+                            int experts, int top, const float* correction, int groups, int keep, int group_best, int renorm,
+                            float scale, int softmax, cudaStream_t stream) {
   if (tokens <= 0) return 0;
   RouteOptions opt;
   if (experts <= 0 || top <= 0 || top > experts || experts > 1024 || stride < experts + (shared_factor ? 1 : 0) ||
-      !route_options(opt, correction, groups, keep, renorm, scale, softmax, experts))
+      !route_options(opt, correction, groups, keep, group_best, renorm, scale, softmax, experts))
     return LB_ERR_SIZE;
   lb_launch(moe_select_kernel, (tokens + SELECT_WARPS - 1) / SELECT_WARPS, SELECT_WARPS * 32,
             (size_t)SELECT_WARPS * (experts + (opt.general() ? experts + opt.groups : 0)) * sizeof(float), stream, logits, stride, ids,

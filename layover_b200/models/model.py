@@ -35,6 +35,8 @@ class Model:
             raise ValueError("adding the embedding output between passes needs a 32-bit residual stream")
         if spec.position_table and spec.residual_dtype != "float32":
             raise ValueError("learned position vectors are added into a 32-bit residual stream")
+        if spec.streams and (spec.residual_dtype != "float32" or self._keeps_embedding):
+            raise ValueError("several residual streams are 32-bit and take no embedding output between passes")
         self.positions = None
 
     # ---- weights
@@ -119,6 +121,8 @@ class Model:
         if self.positions is not None:      # a learned vector per position, unscaled
             ops.add_position_rows(x, batch.positions, self.positions)
         embedded = x.clone() if self._keeps_embedding else None     # the stream is updated in place
+        if self.spec.streams:           # the streams start out equal: one row stands for all of a token's
+            x = x[:, None, :].expand(-1, self.spec.streams, -1)
         delta = None
         for index, entry in enumerate(self.spec.schedule):
             with profiling.nvtx_range(self._range_names[index]) if profiling.active() else _NO_RANGE:

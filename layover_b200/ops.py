@@ -212,14 +212,14 @@ def qk_rownorm_kv(proj: torch.Tensor, q_out: torch.Tensor, k_pool: torch.Tensor,
               q_room, k_room, v_room, _stream()), "qk_rownorm_kv")
 
 
-def rope_table(positions: torch.Tensor, inv_freq: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
-    """out[t, 0, i] = cos(positions[t] * inv_freq[i]), out[t, 1, i] = sin(...); out float32 [T, 2, n_freq]."""
+def rope_table(positions: torch.Tensor, inv_freq: torch.Tensor, out: torch.Tensor, amplitude: float = 1.0) -> torch.Tensor:
+    """out[t, 0, i] = amplitude cos(positions[t] * inv_freq[i]), out[t, 1, i] = amplitude sin(...); out float32 [T, 2, n_freq]."""
     _need(positions, torch.int32, "positions"); _need(inv_freq, torch.float32, "inv_freq"); _need(out, torch.float32, "out")
     tokens, n_freq = positions.shape[0], inv_freq.shape[0]
     if tuple(out.shape) != (tokens, 2, n_freq):
         raise ValueError("rope_table: out must be [tokens, 2, n_freq]")
-    fn = _fn("elementwise", "lb_rope_table", [c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p])
-    _check(fn(_ptr(positions), _ptr(inv_freq), _ptr(out), tokens, n_freq, _stream()), "rope_table")
+    fn = _fn("elementwise", "lb_rope_table", [c_void_p, c_void_p, c_void_p, c_int, c_int, c_float, c_void_p])
+    _check(fn(_ptr(positions), _ptr(inv_freq), _ptr(out), tokens, n_freq, float(amplitude), _stream()), "rope_table")
     return out
 
 
@@ -328,7 +328,8 @@ def heads_bias_rope_kv(proj: torch.Tensor, q_out: torch.Tensor, k_pool: torch.Te
                        blend_weight: torch.Tensor | None, q_heads: int, kv_heads: int, dim: int, vdim: int,
                        page_tokens: int, q_norm_w: torch.Tensor | None = None, k_norm_w: torch.Tensor | None = None,
                        norm_eps: float = 0.0, neighbours: bool = False, values_from_keys: bool = False,
-                       temperature: tuple[float, int] | None = None, positions: torch.Tensor | None = None) -> None:
+                       temperature: tuple[float, int] | None = None, positions: torch.Tensor | None = None,
+                       whole_norm: bool = False) -> None:
     """Biases, a rotation of the first channels of every q and k head, an optional blend of the values with an
     earlier layer's, q to q_out and k, v to their pages.
 
@@ -341,7 +342,8 @@ def heads_bias_rope_kv(proj: torch.Tensor, q_out: torch.Tensor, k_pool: torch.Te
     weight and `norm_eps`, after the biases and before the rotation. `neighbours`: channels 2i and 2i + 1 turn together
     (i < n_freq) instead of i and i + n_freq. `values_from_keys`: the row holds no values; a value head is its key head as
     projected (with the key's bias), before norm and rotation, so vdim = dim. `temperature` = (coef, every): q is also
-    multiplied by 1 + coef ln(floor((p + 1) / every) + 1) at position p = positions[t] (int32 [T])."""
+    multiplied by 1 + coef ln(floor((p + 1) / every) + 1) at position p = positions[t] (int32 [T]). `whole_norm`: q is normed over
+    all its heads at once and so is k, with weights q_norm_w [q_heads * dim] and k_norm_w [kv_heads * dim]."""
     _need_rows(proj, torch.float32, "proj"); _need(k_pool, q_out.dtype, "k_pool"); _need(v_pool, q_out.dtype, "v_pool")
     _need(q_out, None, "q_out"); _need(slot_map, torch.int32, "slot_map")
     tokens = proj.shape[0]
@@ -375,11 +377,12 @@ def heads_bias_rope_kv(proj: torch.Tensor, q_out: torch.Tensor, k_pool: torch.Te
         _need(blend_weight, torch.float32, "blend_weight")
         if blend_weight.numel() != 1:
             raise ValueError("heads_bias_rope_kv: blend_weight is one number")
-    for name, t in (("q_norm_w", q_norm_w), ("k_norm_w", k_norm_w)):
+    for name, t, heads in (("q_norm_w", q_norm_w, q_heads), ("k_norm_w", k_norm_w, kv_heads)):
+        entries = heads * dim if whole_norm else dim
         if t is not None:
             _need(t, torch.float32, name)
-            if t.numel() != dim:
-                raise ValueError(f"heads_bias_rope_kv: {name} must have {dim} entries")
+            if t.numel() != entries:
+                raise ValueError(f"heads_bias_rope_kv: {name} must have {entries} entries")
     coef, every = (float(temperature[0]), int(temperature[1])) if temperature is not None else (0.0, 0)
     if temperature is not None:
         _need(positions, torch.int32, "positions")
@@ -391,7 +394,7 @@ def heads_bias_rope_kv(proj: torch.Tensor, q_out: torch.Tensor, k_pool: torch.Te
     _check(fn(dtype_code(q_out.dtype), _ptr(proj), proj.stride(0), _ptr(q_out), _ptr(k_pool), _ptr(v_pool), _ptr(q_bias),
               _ptr(k_bias), _ptr(v_bias), _ptr(table), n_freq, _ptr(slot_map), _ptr(first_v if blend else None), int(blend),
               _ptr(blend_weight if blend == 2 else None), tokens, q_heads, kv_heads, dim, vdim, page_tokens, q_room, k_room,
-              v_room, _ptr(q_norm_w), _ptr(k_norm_w), float(norm_eps), (1 if neighbours else 0) | (2 if values_from_keys else 0),
+              v_room, _ptr(q_norm_w), _ptr(k_norm_w), float(norm_eps), (1 if neighbours else 0) | (2 if values_from_keys else 0) | (4 if whole_norm else 0),
               _ptr(positions if every else None), coef, every, _stream()), "heads_bias_rope_kv")
 
 
@@ -434,10 +437,12 @@ def softcap(logits: torch.Tensor, cap: float) -> torch.Tensor:
 
 # ------------------------------------------------------------------ routed experts
 EXPERT_ACTIVATIONS = {"silu": 0, "relu": 1, "relu2": 2, "clipped_swiglu": 3}
-ROUTE_SCORES = {"sigmoid": 0, "softmax": 1}     # of a chosen expert's logit alone, or over the chosen logits
+# of a chosen expert's logit alone, over the chosen logits, or over all experts' logits
+ROUTE_SCORES = {"sigmoid": 0, "softmax": 1, "softmax_all": 2}
+GROUP_SCORES = ("two_best", "best")             # a group's score: the sum of its two largest choice scores, or the largest
 
 
-def _route_options(experts: int, correction, groups, keep_groups, renormalize, route_scale, score, what: str):
+def _route_options(experts: int, correction, groups, keep_groups, group_score, renormalize, route_scale, score, what: str):
     """The router's further options as the kernels take them (see `moe_route`)."""
     groups = int(groups or 0)
     keep = int(keep_groups or groups or 0)
@@ -449,17 +454,17 @@ def _route_options(experts: int, correction, groups, keep_groups, renormalize, r
         raise ValueError(f"{what}: the experts must form equal groups of which 1..groups are kept")
     if not float(route_scale) > 0:
         raise ValueError(f"{what}: route_scale must be positive")
-    if score not in ROUTE_SCORES:
-        raise ValueError(f"{what}: unknown score {score!r}")
+    if score not in ROUTE_SCORES or group_score not in GROUP_SCORES:
+        raise ValueError(f"{what}: unknown score {score!r} or group score {group_score!r}")
     if score == "softmax" and (correction is not None or groups > 1 or renormalize or float(route_scale) != 1.0):
         raise ValueError(f"{what}: softmax weights do not combine with corrections, groups, renormalisation or a scale")
-    return [_ptr(correction), groups, keep, int(bool(renormalize)), float(route_scale), ROUTE_SCORES[score]]
+    return [_ptr(correction), groups, keep, int(group_score == "best"), int(bool(renormalize)), float(route_scale), ROUTE_SCORES[score]]
 
 
 def moe_route(h: torch.Tensor, router: torch.Tensor, top: int, ids: torch.Tensor, scores: torch.Tensor,
               shared_w: torch.Tensor | None = None, shared_factor: torch.Tensor | None = None,
               correction: torch.Tensor | None = None, groups: int | None = None, keep_groups: int | None = None,
-              renormalize: bool = False, route_scale: float = 1.0, score: str = "sigmoid") -> None:
+              renormalize: bool = False, route_scale: float = 1.0, score: str = "sigmoid", group_score: str = "two_best") -> None:
     """ids[t, k], scores[t, k]: the `top` experts with the largest router logits of token t (ties: the lower index) and
     sigmoid of those logits. h [T, H] in the run's type; router float32 [experts, H]; logits are 32-bit dot products.
     `shared_w` float32 [H]: also shared_factor[t] = sigmoid(shared_w . h[t]).
@@ -467,7 +472,8 @@ def moe_route(h: torch.Tensor, router: torch.Tensor, top: int, ids: torch.Tensor
     the experts form that many equal groups of neighbours, a group's score is the sum of its two largest choice scores,
     and only experts of the `keep_groups` best groups can be chosen. `renormalize`: the chosen scores are divided by their
     sum (+ 1e-20); `route_scale` then multiplies them. `score` "softmax": the scores are the softmax over the chosen logits
-    (and none of the further options apply)."""
+    (and none of the further options apply); "softmax_all": a score is the softmax over all experts' logits instead of the
+    sigmoid of its own. `group_score` "best": a group's score is its largest choice score alone."""
     _need(h, None, "h"); _need(router, torch.float32, "router"); _need(ids, torch.int32, "ids"); _need(scores, torch.float32, "scores")
     tokens, hidden = h.shape
     experts = router.shape[0]
@@ -477,15 +483,16 @@ def moe_route(h: torch.Tensor, router: torch.Tensor, top: int, ids: torch.Tensor
         _need(shared_w, torch.float32, "shared_w"); _need(shared_factor, torch.float32, "shared_factor")
         if shared_w.numel() != hidden or shared_factor.numel() != tokens:
             raise ValueError("moe_route: shared_w [H] and shared_factor [T]")
-    options = _route_options(experts, correction, groups, keep_groups, renormalize, route_scale, score, "moe_route")
-    fn = _fn("moe", "lb_moe_route", [c_int] + [c_void_p] * 6 + [c_int] * 4 + [c_void_p, c_int, c_int, c_int, c_float, c_int, c_void_p])
+    options = _route_options(experts, correction, groups, keep_groups, group_score, renormalize, route_scale, score, "moe_route")
+    fn = _fn("moe", "lb_moe_route", [c_int] + [c_void_p] * 6 + [c_int] * 4 + [c_void_p, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p])
     _check(fn(dtype_code(h.dtype), _ptr(h), _ptr(router), _ptr(shared_w), _ptr(ids), _ptr(scores), _ptr(shared_factor), tokens,
               hidden, experts, int(top), *options, _stream()), "moe_route")
 
 
 def moe_select(logits: torch.Tensor, experts: int, top: int, ids: torch.Tensor, scores: torch.Tensor,
                shared_factor: torch.Tensor | None = None, correction: torch.Tensor | None = None, groups: int | None = None,
-               keep_groups: int | None = None, renormalize: bool = False, route_scale: float = 1.0, score: str = "sigmoid") -> None:
+               keep_groups: int | None = None, renormalize: bool = False, route_scale: float = 1.0, score: str = "sigmoid",
+               group_score: str = "two_best") -> None:
     """What `moe_route` chooses, from router logits that a matrix product left in float32 [T, >= experts (+ 1)]: the
     `top` largest of the first `experts` columns (ties: the lower index), their sigmoids, and, with `shared_factor`,
     sigmoid of column `experts`."""
@@ -496,9 +503,9 @@ def moe_select(logits: torch.Tensor, experts: int, top: int, ids: torch.Tensor, 
         raise ValueError("moe_select: shapes do not agree")
     if shared_factor is not None:
         _need(shared_factor, torch.float32, "shared_factor")
-    options = _route_options(experts, correction, groups, keep_groups, renormalize, route_scale, score, "moe_select")
+    options = _route_options(experts, correction, groups, keep_groups, group_score, renormalize, route_scale, score, "moe_select")
     fn = _fn("moe", "lb_moe_select", [c_void_p, c_long, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
-                                      c_void_p, c_int, c_int, c_int, c_float, c_int, c_void_p])
+                                      c_void_p, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p])
     _check(fn(_ptr(logits), logits.stride(0), _ptr(ids), _ptr(scores), _ptr(shared_factor), tokens, int(experts), int(top),
               *options, _stream()), "moe_select")
 
@@ -613,7 +620,7 @@ def moe_scatter_rows(h: torch.Tensor, place_of: torch.Tensor, scale: torch.Tenso
     return rows
 
 
-GROUPED_EPILOGUES = {None: 0, "swiglu": 1, "clipped_swiglu": 3}
+GATED_EPILOGUES = {None: 0, "swiglu": 1, "clipped_swiglu": 3}
 
 
 def gemm_tcgen05_grouped(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, tile_rows: torch.Tensor, groups: int,
@@ -629,7 +636,7 @@ def gemm_tcgen05_grouped(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, ti
     if w.shape[0] % groups or w.shape[1] != k or m % MOE_TILE_ROWS:
         raise ValueError("gemm_tcgen05_grouped: shapes do not agree")
     n = w.shape[0] // groups
-    if epilogue not in GROUPED_EPILOGUES:
+    if epilogue not in GATED_EPILOGUES:
         raise ValueError(f"gemm_tcgen05_grouped: unknown epilogue {epilogue!r}")
     out_cols = n // 2 if epilogue else n
     if epilogue and (n % (2 * SWIGLU_BLOCK) or out.dtype != torch.bfloat16):
@@ -643,7 +650,68 @@ def gemm_tcgen05_grouped(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, ti
               c_void_p, c_int, c_int, c_int, c_float, c_float, c_void_p])
     _check(fn(_ptr(a), _ptr(w), _ptr(out), dtype_code(out.dtype), m, n, k, int(groups), a.stride(0), w.stride(0), out.stride(0),
               _ptr(tile_rows), _ptr(partials), partials.numel(), _ptr(counters), counters.numel(), sms,
-              GROUPED_EPILOGUES[epilogue], float(limit), float(slope), _stream()), "gemm_tcgen05_grouped")
+              GATED_EPILOGUES[epilogue], float(limit), float(slope), _stream()), "gemm_tcgen05_grouped")
+    return out
+
+
+# ------------------------------------------------------------------ several residual streams
+def stream_shift_tokens() -> int:
+    lib = build.load("streams")
+    lib.lb_stream_shift_tokens.restype = c_int
+    return lib.lb_stream_shift_tokens()
+
+
+def stream_norm(x: torch.Tensor, update: tuple | None, read: torch.Tensor | None, weight: torch.Tensor, eps: float,
+                out: torch.Tensor, x_out: torch.Tensor | None = None, rows: torch.Tensor | None = None,
+                shift: tuple | None = None) -> torch.Tensor:
+    """What happens to several residual streams between two sub-layers, in one kernel, all of it 32-bit:
+
+        x'_t = sum_s mix[s, t] x_s + gain[t] y,     h = weight * norm(sum_t read[t] x'_t)
+
+    x float32 [T, S, W] (a token's streams may be one row, stride 0); `update` = (y [T, W] in the run's type, mix float32
+    [S, S], gain float32 [S]) or None: x' = x. read float32 [S], or None: the plain sum. x_out float32 [T, S, W], another
+    buffer than x, receives x' (None: nobody needs it). out [T, W] in the run's type receives h; with `rows` (int32) only
+    the listed tokens' h, in that order. `shift` = (mu float32 [W], state float32 [slots, >= W], batch): out is h + (h_before
+    - h) * mu instead, h_before the unrounded h of the sequence's previous token (its state row at the start of the step;
+    the step's last h is left there)."""
+    _need(weight, torch.float32, "weight"); _need(out, None, "out")
+    if x.dim() != 3 or x.dtype != torch.float32 or x.stride(2) != 1:
+        raise ValueError("stream_norm: x must be float32 [tokens, streams, width]")
+    tokens, streams, width = x.shape
+    blocks = tokens if rows is None else rows.shape[0]
+    if weight.numel() != width or tuple(out.shape) != (blocks, width):
+        raise ValueError("stream_norm: weight [width] and a row of out per token")
+    y = mix = gain = None
+    if update is not None:
+        y, mix, gain = update
+        _need(y, out.dtype, "y"); _need(mix, torch.float32, "mix"); _need(gain, torch.float32, "gain")
+        if tuple(y.shape) != (tokens, width) or tuple(mix.shape) != (streams, streams) or gain.numel() != streams:
+            raise ValueError("stream_norm: the update is y [tokens, width], mix [streams, streams], gain [streams]")
+    if read is not None:
+        _need(read, torch.float32, "read")
+        if read.numel() != streams:
+            raise ValueError("stream_norm: read must have one weight per stream")
+    if x_out is not None:
+        _need(x_out, torch.float32, "x_out")
+        if tuple(x_out.shape) != tuple(x.shape) or x_out.data_ptr() == x.data_ptr() or rows is not None:
+            raise ValueError("stream_norm: x_out is another [tokens, streams, width] buffer than x, and has no picked rows")
+    if rows is not None:
+        _need(rows, torch.int32, "rows")
+    mu = state = tiles = batch = None
+    if shift is not None:
+        mu, state, batch = shift
+        _need(mu, torch.float32, "mu"); _need(state, torch.float32, "state")
+        if mu.numel() != width or state.dim() != 2 or state.shape[1] < width or rows is not None or batch.n_tokens != tokens:
+            raise ValueError("stream_norm: the shift is mu [width], state [slots, >= width] and this batch, without picked rows")
+        tiles = batch.tiles[stream_shift_tokens()]
+        blocks = tiles.count
+    fn = _fn("streams", "lb_stream_norm", [c_int, c_void_p, c_long, c_long] + [c_void_p] * 6 + [c_float, c_void_p, c_void_p, c_int, c_int, c_int,
+                                           c_void_p, c_void_p, c_long] + [c_void_p] * 5)
+    _check(fn(dtype_code(out.dtype), _ptr(x), x.stride(0), x.stride(1), _ptr(y), _ptr(mix), _ptr(gain), _ptr(read), _ptr(x_out),
+              _ptr(weight), float(eps), _ptr(out), _ptr(rows), blocks, width, streams, _ptr(mu), _ptr(state),
+              state.stride(0) if state is not None else 0, _ptr(batch.cu_q if batch is not None else None),
+              _ptr(batch.state_slots if batch is not None else None), _ptr(tiles.tile_seq if tiles else None),
+              _ptr(tiles.tile_q0 if tiles else None), _stream()), "stream_norm")
     return out
 
 
@@ -784,53 +852,71 @@ def scaled_add_rmsnorm(x: torch.Tensor, a: torch.Tensor | None, a_weight: torch.
 
 
 # ------------------------------------------------------------------ attention over a latent
-def latent_rows(proj: torch.Tensor, q_off: int, dkv_off: int, norm_w: torch.Tensor | None, eps: float, table: torch.Tensor,
-                slot_map: torch.Tensor | None, k_pool: torch.Tensor | None, q_out: torch.Tensor, q_heads: int, dim: int,
-                rot: int, rank: int, page_tokens: int) -> None:
+def latent_rows(proj: torch.Tensor, dkv_off: int, norm_w: torch.Tensor | None, eps: float, table: torch.Tensor | None,
+                slot_map: torch.Tensor | None, k_pool: torch.Tensor | None, rot: int, rank: int, page_tokens: int,
+                cq_off: int = 0, cq_norm_w: torch.Tensor | None = None, cq_out: torch.Tensor | None = None) -> None:
     """A token's cache row [normed latent | rotated key part | zeros] into `k_pool` [pages, 1, page_tokens, room] (not with
-    dkv_off < 0: a layer that reads another layer's rows), and the rotated part of every query head into channels
-    [rank, rank + rot) of q_out [T, q_heads * room] (zeros behind it; channels [0, rank) are left alone).
-    proj float32 rows: q_heads x [dim | rot] at q_off, [rank | rot] at dkv_off; table float32 [T, 2, rot / 2] from
-    `rope_table`: channels 2i and 2i + 1 of a rotated part turn by angle i."""
-    _need(proj, torch.float32, "proj"); _need(table, torch.float32, "table"); _need(q_out, None, "q_out")
-    tokens = proj.shape[0]
-    room = q_out.shape[1] // q_heads
-    if proj.dim() != 2 or proj.stride(1) != 1 or q_out.shape[0] != tokens or q_out.shape[1] != q_heads * room or room < rank + rot:
-        raise ValueError("latent_rows: q_out must be [tokens, q_heads * room] with room >= rank + rot")
-    if tuple(table.shape) != (tokens, 2, rot // 2) or rot % 2:
-        raise ValueError("latent_rows: the rotary table must be [tokens, 2, rot / 2]")
+    dkv_off < 0: a layer that reads another layer's rows), and, with `cq_out` [T, cq_rank], the normed latent of the queries.
+    proj float32 rows: [rank | rot] at dkv_off, cq_rank channels at cq_off; table float32 [T, 2, rot / 2] from
+    `rope_table`: channels 2i and 2i + 1 of the rotated part turn by angle i."""
+    _need(proj, torch.float32, "proj")
+    tokens, room, cq_rank = proj.shape[0], 0, 0
     if dkv_off >= 0:
-        _need(norm_w, torch.float32, "norm_w"); _need(slot_map, torch.int32, "slot_map"); _need(k_pool, q_out.dtype, "k_pool")
-        if norm_w.numel() != rank or tuple(k_pool.shape[1:]) != (1, page_tokens, room):
-            raise ValueError("latent_rows: the pool must be [pages, 1, page_tokens, room] and the norm weight [rank]")
-    fn = _fn("latent", "lb_latent_rows", [c_int, c_void_p, c_long, c_int, c_int, c_void_p, c_float, c_void_p, c_void_p, c_void_p,
-                                          c_void_p] + [c_int] * 7 + [c_void_p])
-    _check(fn(dtype_code(q_out.dtype), _ptr(proj), proj.stride(0), int(q_off), int(dkv_off), _ptr(norm_w), float(eps), _ptr(table),
-              _ptr(slot_map), _ptr(k_pool), _ptr(q_out), tokens, q_heads, dim, rot, rank, room, page_tokens, _stream()),
+        _need(norm_w, torch.float32, "norm_w"); _need(slot_map, torch.int32, "slot_map"); _need(k_pool, None, "k_pool")
+        _need(table, torch.float32, "table")
+        room = k_pool.shape[-1]
+        if norm_w.numel() != rank or tuple(k_pool.shape[1:]) != (1, page_tokens, room) or room < rank + rot:
+            raise ValueError("latent_rows: the pool must be [pages, 1, page_tokens, room >= rank + rot] and the norm weight [rank]")
+        if tuple(table.shape) != (tokens, 2, rot // 2) or rot % 2:
+            raise ValueError("latent_rows: the rotary table must be [tokens, 2, rot / 2]")
+        if proj.shape[1] < dkv_off + rank + rot:
+            raise ValueError("latent_rows: the projection row does not hold the latent")
+    if cq_out is not None:
+        _need(cq_out, k_pool.dtype if dkv_off >= 0 else None, "cq_out"); _need(cq_norm_w, torch.float32, "cq_norm_w")
+        cq_rank = cq_out.shape[1]
+        if cq_out.shape[0] != tokens or cq_norm_w.numel() != cq_rank or not 0 <= cq_off <= proj.shape[1] - cq_rank:
+            raise ValueError("latent_rows: the projection row does not hold the queries' latent")
+    dtype = (k_pool if dkv_off >= 0 else cq_out).dtype
+    fn = _fn("latent", "lb_latent_rows", [c_int, c_void_p, c_long, c_int, c_void_p, c_float, c_void_p, c_void_p, c_void_p] + [c_int] * 7
+             + [c_void_p, c_void_p, c_void_p])
+    _check(fn(dtype_code(dtype), _ptr(proj), proj.stride(0), int(dkv_off), _ptr(norm_w), float(eps), _ptr(table), _ptr(slot_map),
+              _ptr(k_pool), tokens, rot, rank, room, page_tokens, int(cq_off), cq_rank, _ptr(cq_norm_w), _ptr(cq_out), _stream()),
            "latent_rows")
 
 
-def heads_linear(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, gate: torch.Tensor | None = None) -> torch.Tensor:
+def heads_linear(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, gate: torch.Tensor | None = None,
+                 tail: tuple[torch.Tensor, int] | None = None) -> torch.Tensor:
     """out[t, h, :] = a[t, h, :] @ w[h]^T, one product per head: a [T, heads, K] and out [T, heads, N] may be views into wider
     rows (the last axis contiguous), w [heads, N, K] dense. a is of w's type, or float32 (unrounded projection rows); out of
-    w's type. `gate` float32 [T, heads * N] (a view into wider rows is fine): out *= sigmoid(gate). 32-bit sums in the
-    order of K."""
+    w's type. `gate` float32 [T, heads * N] or, one per head, [T, heads] (a view into wider rows is fine): out *=
+    sigmoid(gate). 32-bit sums in the order of K. `tail` = (table, rot): a is [T, heads, K + rot] and out [T, heads, room]; the
+    last rot channels of a head are turned (channels 2i and 2i + 1 by angle i of `rope_table`'s table [T, 2, rot / 2]) and
+    follow the N outputs, zeros behind them."""
     _need(w, None, "w")
     tokens, heads, k_dim = a.shape
-    n_out = w.shape[1]
-    if w.dim() != 3 or w.shape[0] != heads or w.shape[2] != k_dim or not w.is_contiguous() or tuple(out.shape) != (tokens, heads, n_out):
+    n_out, table, rot, tail_room = w.shape[1], None, 0, 0
+    if tail is not None:
+        table, rot = tail[0], int(tail[1])
+        k_dim, tail_room = k_dim - rot, out.shape[2] - n_out
+        _need(table, torch.float32, "table")
+        if tuple(table.shape) != (tokens, 2, rot // 2) or rot % 2 or tail_room < rot:
+            raise ValueError("heads_linear: the rotary table must be [tokens, 2, rot / 2] and out hold N + rot channels a head")
+    if w.dim() != 3 or w.shape[0] != heads or w.shape[2] != k_dim or not w.is_contiguous() \
+            or tuple(out.shape) != (tokens, heads, n_out + tail_room):
         raise ValueError("heads_linear: shapes do not agree")
     if a.device != w.device or out.device != w.device or a.stride(2) != 1 or out.stride(2) != 1 or out.dtype != w.dtype \
             or a.dtype not in (w.dtype, torch.float32):
         raise ValueError("heads_linear: a and out must be on the device, contiguous along the last axis, out of w's type")
+    per_head = gate is not None and gate.shape[1] == heads and n_out != 1
     if gate is not None:
-        if gate.dtype != torch.float32 or gate.dim() != 2 or gate.stride(1) != 1 or tuple(gate.shape) != (tokens, heads * n_out):
-            raise ValueError("heads_linear: gate must be [tokens, heads * N]")
+        if gate.dtype != torch.float32 or gate.dim() != 2 or gate.stride(1) != 1 or gate.shape[0] != tokens \
+                or gate.shape[1] not in (heads, heads * n_out):
+            raise ValueError("heads_linear: gate must be [tokens, heads * N] or [tokens, heads]")
     fn = _fn("latent", "lb_heads_linear", [c_int, c_int, c_void_p, c_long, c_long, c_void_p, c_void_p, c_long, c_long, c_void_p,
-                                           c_long, c_int, c_int, c_int, c_int, c_void_p])
+                                           c_long, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int, c_int, c_void_p])
     _check(fn(dtype_code(w.dtype), int(a.dtype == torch.float32), _ptr(a), a.stride(0), a.stride(1), _ptr(w), _ptr(out),
-              out.stride(0), out.stride(1), _ptr(gate), gate.stride(0) if gate is not None else 0, tokens, heads, n_out, k_dim,
-              _stream()), "heads_linear")
+              out.stride(0), out.stride(1), _ptr(gate), gate.stride(0) if gate is not None else 0, int(per_head), tokens, heads, n_out,
+              k_dim, _ptr(table), rot, tail_room, _stream()), "heads_linear")
     return out
 
 
@@ -1216,29 +1302,30 @@ def interleave_gate_up(gate: torch.Tensor, up: torch.Tensor) -> torch.Tensor:
 
 
 def gemm_tcgen05(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, max_splits: int = 0,
-                 epilogue: str | None = None) -> torch.Tensor:
+                 epilogue: str | None = None, limit: float = 0.0, slope: float = 1.0) -> torch.Tensor:
     """out[M, N] = a[M, K] @ w[N, K]^T on the tcgen05 tensor cores; bfloat16 in, out bfloat16 or float32.
 
     epilogue "swiglu": w's rows are interleaved by `interleave_gate_up` and out[M, N / 2] = silu(gate) * up,
-    rounded where the reference's bfloat16 tensors round."""
+    rounded where the reference's bfloat16 tensors round. "clipped_swiglu": the same rows with that activation (see
+    `gated_act`), for up to 16 and for more than 128 rows of `a`."""
     if a.dtype != torch.bfloat16 or w.dtype != torch.bfloat16 or a.dim() != 2 or w.dim() != 2:
         raise ValueError("gemm_tcgen05: operands must be 2-D bfloat16")
     m, k = a.shape
     n = w.shape[0]
-    if epilogue not in (None, "swiglu"):
+    if epilogue not in GATED_EPILOGUES:
         raise ValueError(f"gemm_tcgen05: unknown epilogue {epilogue!r}")
-    out_cols = n // 2 if epilogue == "swiglu" else n
-    if epilogue == "swiglu" and (n % (2 * SWIGLU_BLOCK) or out.dtype != torch.bfloat16):
-        raise ValueError("gemm_tcgen05: the swiglu epilogue needs interleaved weights (2 I rows, I % 64 == 0) and a bfloat16 output")
+    out_cols = n // 2 if epilogue else n
+    if epilogue and (n % (2 * SWIGLU_BLOCK) or out.dtype != torch.bfloat16):
+        raise ValueError(f"gemm_tcgen05: the {epilogue} epilogue needs interleaved weights (2 I rows, I % 64 == 0) and a bfloat16 output")
     if w.shape[1] != k or tuple(out.shape) != (m, out_cols) or out.stride(1) != 1:
         raise ValueError(f"gemm: shapes do not agree: a {tuple(a.shape)}, w {tuple(w.shape)}, out {tuple(out.shape)}")
     partials, counters, sms = gemm_scratch(a.device)
     fn = _fn("gemm_tcgen05", "lb_gemm_tcgen05",
              [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_long, c_long, c_long, c_void_p, c_long,
-              c_void_p, c_int, c_int, c_int, c_int, c_void_p])
+              c_void_p, c_int, c_int, c_int, c_int, c_float, c_float, c_void_p])
     _check(fn(_ptr(a), _ptr(w), _ptr(out), dtype_code(out.dtype), m, n, k, a.stride(0), w.stride(0), out.stride(0),
               _ptr(partials), partials.numel(), _ptr(counters), counters.numel(), sms, int(max_splits),
-              1 if epilogue == "swiglu" else 0, _stream()), "gemm_tcgen05")
+              GATED_EPILOGUES[epilogue], float(limit), float(slope), _stream()), "gemm_tcgen05")
     return out
 
 

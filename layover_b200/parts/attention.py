@@ -57,8 +57,8 @@ class Attention(Part):
     cache are (1 - w) v + w kept values of the same token, w = the scalar tensor `value_blend_weight`).
     With any of these the stacked product leaves 32-bit rows and ONE kernel adds the biases, rotates, blends
     and writes q and the pages (rounded once); a channel gate is one more small kernel after the attention.
-    They do not combine with the whole-row norm or head gates; a norm per head (`qk_norm_eps` with the default
-    `qk_norm`) does: it is applied in the same kernel, after the biases and before the rotation.
+    They do not combine with head gates; a norm per head (`qk_norm_eps` with the default `qk_norm`) or over whole rows
+    (`qk_norm` = "whole") does: it is applied in the same kernel, after the biases and before the rotation.
     `values` = "keys": the layer has no v projection; what a key/value head stores as its value is its raw key
     projection, taken before the key is normed and turned (`v_head_dim` = `head_dim`). A `position` that pairs neighbouring channels (`rotary_pairs`) turns channels 2i
     and 2i + 1 together. Both take this path.
@@ -125,10 +125,10 @@ class Attention(Part):
         self.position = build_part("position", p.get("position"), prefix)
         if self.general and (self.shares_cache or (self.position is not None and not self.rows32)):
             raise ValueError("attention with sinks, head gates, a whole-row norm or its own value size has no rotation "
-                             "and no shared cache")
-        if self.rows32 and ((self.qk_norm_eps is not None and self.qk_norm == "whole") or (p.get("gate") and self.gate_kind == "head")):
+                             "(unless `exact_weights` asks for it) and no shared cache")
+        if self.rows32 and p.get("gate") and self.gate_kind == "head":
             raise ValueError("attention: biases, partial rotation, chunks, value blends and channel gates do not combine "
-                             "with whole-row q/k norms or head gates")
+                             "with head gates")
         if self.chunk and self.window:
             raise ValueError("attention: a window and a chunked mask do not combine")
         if self.chunk < 0:
@@ -300,7 +300,8 @@ class Attention(Part):
                                    self.q_norm_w, self.k_norm_w, float(self.qk_norm_eps or 0.0),
                                    neighbours=getattr(self.position, "pairing", "half") == "neighbours",
                                    values_from_keys=self.values_from_keys, temperature=self.temperature,
-                                   positions=batch.positions if self.temperature is not None else None)
+                                   positions=batch.positions if self.temperature is not None else None,
+                                   whole_norm=self.qk_norm == "whole")
         else:
             if "gate" in self.names:
                 gates = torch.empty((tokens, self.q_heads), dtype=torch.float32, device=out.device)

@@ -3,9 +3,14 @@
 from __future__ import annotations
 
 import contextlib
+import dataclasses
 
-from .. import profiling
-from .base import Part, build_part, register_block
+import torch
+
+from .. import ops, profiling
+from ..weights.loader import TensorSpec
+from .base import Part, StateNeed, build_part, register_block
+from .norm import StreamUpdate
 
 _NO_RANGE = contextlib.nullcontext()
 
@@ -193,8 +198,6 @@ class PostNormBlock(Part):
             return x, None
         held = batch.shared.get(self.LOWERED)
         if held is None or held[0] is not x:
-            import torch
-            from .. import ops
             lowered = torch.empty(x.shape, dtype=self.runtime.dtype, device=x.device)
             ops.lower_rows(x, lowered)
             held = batch.shared[self.LOWERED] = (x, lowered)
@@ -238,3 +241,99 @@ class OutputNormBlock(PostNormBlock):
             with profiling.nvtx_range("feed_forward") if profiling.active() else _NO_RANGE:
                 self.ff_norm.add_normed(x, self.feed_forward.forward(h), self.mult, lowered)
         return x, None
+
+
+@register_block("hyper_connected")
+class HyperConnectedBlock(Part):
+    """Sub-layers around several residual streams x_1 .. x_S instead of one. Each sub-layer reads a weighted sum of the
+    streams, u = sum_s in[s] x_s, y = sub-layer(norm(u)), and then all streams are made anew from the old ones, x_t <-
+    sum_s mix[s, t] x_s + mult * out[t] * y. `connections` = two dicts of tensor names in [S], out [S], mix [S, S] ([from,
+    to]), one for the mixer and one for the feed-forward.
+
+    Nothing is joined here: a sub-layer's output is handed on as a `StreamUpdate` and the next norm of the streams (of this
+    block, of the next one, or the model's final one, which reads their sum) joins it, makes the streams, their weighted
+    sum and its norm in one kernel.
+
+    `shift` (tensor name, [hidden]): what the mixer reads is moved towards what it read at the sequence's token before,
+    element by element: h + (h_before - h) * shift, h_before without a shift of its own and zero before the first token. It
+    is part of a request's state (32-bit, unrounded), beside whatever the mixer keeps, and happens in the same kernel.
+
+    params: streams, hidden, mult, connections, input_norm, mixer (PartSpecs), shift (or None); post_norm, feed_forward
+    (PartSpecs, or both None: a layer without a feed-forward, whose second dict of `connections` is not read)."""
+
+    def __init__(self, params, prefix):
+        super().__init__(params, prefix)
+        self.require("streams", "hidden", "connections", "input_norm", "mixer")
+        self.streams, self.hidden, self.mult = int(params["streams"]), int(params["hidden"]), float(params.get("mult", 1.0))
+        if self.streams < 1:
+            raise ValueError(f"hyper_connected: at least one stream, got {self.streams}")
+        self.input_norm = build_part("norm", params["input_norm"], prefix)
+        self.mixer = build_part("mixer", params["mixer"], prefix)
+        if (params.get("feed_forward") is None) != (params.get("post_norm") is None):
+            raise ValueError("hyper_connected: post_norm and feed_forward come together or not at all")
+        self.post_norm = build_part("norm", params.get("post_norm"), prefix)
+        self.feed_forward = build_part("feed_forward", params.get("feed_forward"), prefix)
+        used = 1 if self.feed_forward is None else 2
+        self.names = [{k: prefix + c[k] for k in ("in", "out", "mix")} for c in params["connections"][:used]]
+        if len(self.names) != used:
+            raise ValueError("hyper_connected: connections for every sub-layer")
+        self.shift_name = prefix + params["shift"] if params.get("shift") else None
+        self.shift = None
+        self.connections = []       # once bound, per sub-layer: (in, mult * out, mix), 32-bit
+
+    def parts(self):
+        return [p for p in (self.input_norm, self.mixer, self.post_norm, self.feed_forward) if p is not None]
+
+    def tensor_specs(self):
+        specs = [spec for part in self.parts() for spec in part.tensor_specs()]
+        for n in self.names:
+            specs += [TensorSpec(n["in"], (self.streams,), kind="vector", init="ones"),
+                      TensorSpec(n["out"], (self.streams,), kind="vector", init="ones"),
+                      TensorSpec(n["mix"], (self.streams, self.streams), kind="vector", init="eye")]
+        if self.shift_name:
+            specs.append(TensorSpec(self.shift_name, (self.hidden,), kind="vector", init="ones", init_offset=-0.5))
+        return specs
+
+    def bind(self, tensors, runtime):
+        super().bind(tensors, runtime)
+        for part in self.parts():
+            part.bind(tensors, runtime)
+        self.connections = [(tensors[n["in"]], self.mult * tensors[n["out"]], tensors[n["mix"]].contiguous()) for n in self.names]
+        self.shift = tensors[self.shift_name] if self.shift_name else None
+
+    def cache_need(self):
+        need = self.mixer.cache_need()
+        if not self.shift_name:
+            return need
+        needs = () if need is None else need if isinstance(need, (tuple, list)) else (need,)
+        return (*needs, StateNeed((self.hidden,), torch.float32))
+
+    def _views(self, cache):
+        """(the mixer's view, the state row of the shift): a block with a shift has a composite view, the shift's last."""
+        if not self.shift_name:
+            return cache, None
+        *views, shift = cache.parts
+        if isinstance(self.mixer.cache_need(), (tuple, list)):
+            return dataclasses.replace(cache, parts=views), shift.state
+        return (views[0] if views else None), shift.state
+
+    def kernel_libraries(self, dtype):
+        return ("streams",)
+
+    def tile_sizes(self, dtype):
+        return (ops.stream_shift_tokens(),) if self.shift_name else ()
+
+    def forward(self, x, delta, batch, cache, extra=None):
+        if extra is not None or x.dim() != 3:
+            raise ValueError("hyper_connected: the residual streams are [tokens, streams, hidden], and nothing else is added to them")
+        view, state = self._views(cache)
+        with profiling.nvtx_range("mixer") if profiling.active() else _NO_RANGE:
+            read, gain, mix = self.connections[0]
+            x, h = self.input_norm.read_streams(x, delta, read, shift=(self.shift, state, batch) if self.shift_name else None)
+            delta = StreamUpdate(self.mixer.forward(h, batch, view), mix, gain)
+        if self.feed_forward is None:
+            return x, delta
+        with profiling.nvtx_range("feed_forward") if profiling.active() else _NO_RANGE:
+            read, gain, mix = self.connections[1]
+            x, h = self.post_norm.read_streams(x, delta, read)
+            return x, StreamUpdate(self.feed_forward.forward(h), mix, gain)

@@ -8,6 +8,9 @@ from .. import ops
 from ..weights.loader import TensorSpec
 from .base import Part, build_part, register_feed_forward
 
+# gated activations that the tensor-core products have as an epilogue, and its name there
+FUSED_ACTIVATIONS = {"silu": "swiglu", "clipped_swiglu": "clipped_swiglu"}
+
 
 @register_feed_forward("gated_mlp")
 class GatedMLP(Part):
@@ -18,7 +21,7 @@ class GatedMLP(Part):
     product reads x once. In a bfloat16 run whose width allows it, the rows are interleaved for
     the tensor-core product with the activation in its epilogue and no [T, 2 inter] tensor is ever
     written; otherwise the activation kernel reads both halves of its row. The product's epilogue
-    knows silu only: with relu the interleaved product is followed by the activation kernel."""
+    knows silu and the clipped gate: with the others the interleaved product is followed by the activation kernel."""
 
     def __init__(self, params, prefix):
         super().__init__(params, prefix)
@@ -54,13 +57,14 @@ class GatedMLP(Part):
         return ("elementwise",)
 
     def activated(self, h: torch.Tensor) -> torch.Tensor:
-        """silu(h Wg^T) * (h Wu^T) over the interleaved weights. Many tokens, or at most 16: one
+        """act(h Wg^T) * (h Wu^T) over the interleaved weights. Many tokens, or at most 16: one
         product with the activation in its epilogue. In between: product, then the activation kernel,
         which is faster there (a whole feed-forward at 64 tokens: 41.7 us against 43.5 us fused)."""
         tokens = h.shape[0]
         out = torch.empty((tokens, self.inter), dtype=torch.bfloat16, device=h.device)
-        if self.activation == "silu" and (tokens > 128 or tokens <= 16) and ops.gemm_tcgen05_supports(h, self.gate_up):
-            return ops.gemm_tcgen05(h, self.gate_up, out, epilogue="swiglu")
+        epilogue = FUSED_ACTIVATIONS.get(self.activation)
+        if epilogue and (tokens > 128 or tokens <= 16) and ops.gemm_tcgen05_supports(h, self.gate_up):
+            return ops.gemm_tcgen05(h, self.gate_up, out, epilogue=epilogue, **self._clip)
         gate_up = self.runtime.linear(h, self.gate_up)
         if self.activation == "silu":
             return ops.swiglu(gate_up, out, block=ops.SWIGLU_BLOCK)
@@ -125,7 +129,9 @@ class RoutedExperts(Part):
     tensor of one number per expert, added to the sigmoids for the choice only), limited to the `keep_groups` best of
     `groups` equal groups of neighbouring experts (a group's score: the sum of its two largest corrected scores), and the
     chosen scores may be divided by their sum (`renormalize`) and multiplied by `route_scale`. `score` = "softmax": the
-    choice is made on the logits and the scores are the softmax over the chosen logits (none of the former apply).
+    choice is made on the logits and the scores are the softmax over the chosen logits (none of the former apply);
+    "softmax_all": the scores are the softmax over all experts' logits, and all of the former apply. `group_score` "best":
+    a group's score is its largest choice score alone (default "two_best").
     `activation` "clipped_swiglu" (with `limit`, `slope`): expert(x) = down(g sigmoid(slope g) (u + 1)), g = min(gate x,
     limit), u = up x within +- limit. On the device:
     route (one warp per token) -> group the (token, expert) pairs by expert -> one launch for all experts'
@@ -147,7 +153,7 @@ class RoutedExperts(Part):
     params: hidden, experts, top, inter, activation ("silu"), router (tensor name), expert_gate / expert_up /
     expert_down (tensor names with `{}` for the expert's index), shared (a feed-forward PartSpec or None),
     shared_gate (tensor name of a [1, hidden] matrix, or None: the shared expert is added as it is); optional gated,
-    score, limit, slope, weight_on, correction (tensor name), groups, keep_groups, renormalize, route_scale."""
+    score, limit, slope, weight_on, correction (tensor name), groups, keep_groups, group_score, renormalize, route_scale."""
 
     def __init__(self, params, prefix):
         super().__init__(params, prefix)
@@ -178,6 +184,9 @@ class RoutedExperts(Part):
                                 or self.keep_groups * (self.experts // self.groups) < self.top):
             raise ValueError(f"routed_experts: {self.experts} experts in {self.groups} groups of which {self.keep_groups} are kept "
                              f"cannot give a token {self.top} experts")
+        self.group_score = p.get("group_score", "two_best")
+        if self.group_score not in ops.GROUP_SCORES:
+            raise ValueError(f"routed_experts: unknown group_score {self.group_score!r}")
         if self.score == "softmax" and (p.get("correction") or self.groups > 1 or self.renormalize or self.route_scale != 1.0):
             raise ValueError("routed_experts: softmax scores do not combine with corrections, groups, renormalisation or a scale")
         self.correction_name = prefix + p["correction"] if p.get("correction") else None
@@ -212,11 +221,11 @@ class RoutedExperts(Part):
         self.router = tensors[self.router_name]
         self.correction = tensors[self.correction_name] if self.correction_name else None
         self._route = dict(correction=self.correction, groups=self.groups, keep_groups=self.keep_groups,
-                           renormalize=self.renormalize, route_scale=self.route_scale, score=self.score)
+                           renormalize=self.renormalize, route_scale=self.route_scale, score=self.score, group_score=self.group_score)
         self._clip = dict(limit=self.limit, slope=self.slope)
         # one copy of the experts' weights serves both forms: where the tensor-core product can fuse the activation
         # (bfloat16, silu or the clipped gate, widths in blocks of 64) every expert's gate and up rows are interleaved for it
-        self.epilogue = {"silu": "swiglu", "clipped_swiglu": "clipped_swiglu"}.get(self.activation)
+        self.epilogue = FUSED_ACTIVATIONS.get(self.activation)
         self.interleaved = (self.gated and runtime.dtype == torch.bfloat16 and self.epilogue is not None
                             and self.inter % ops.SWIGLU_BLOCK == 0)
         stack = ops.interleave_gate_up if self.interleaved else (lambda gate, up: torch.cat((gate, up), dim=0))

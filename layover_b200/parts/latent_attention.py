@@ -25,11 +25,16 @@ class LatentAttention(Part):
     W_uv,h with the gate in the same kernel. A layer with `shares_cache` has no W_down: it reads the rows of
     an earlier layer (the schedule names it) through maps of its own.
 
+    With `q_rank` the queries come from a latent of their own: q = W_uq rmsnorm(W_dq h) (tensors `q_down` [q_rank, hidden],
+    `q_down_norm`, and `q` [heads * (dim + rot_dim), q_rank]); W_dq's rows join the stacked product, the kernel that makes
+    the cache rows norms them too, and W_uq is a product of its own. `gate_kind` = "head": W_g is [heads, hidden] and head
+    h's output is multiplied by sigmoid(W_g h)_h (default "channel").
+
     params: hidden, heads, head_dim (unrotated), rot_dim, v_head_dim, kv_rank, scale, norm_eps, position (a
     PartSpec over rot_dim channels whose table the kernel applies to neighbouring pairs), shares_cache; window (None:
     every earlier token) and cache_window (the window the cached rows are kept for: the widest of this layer's and of
-    the layers' that read its rows; default: window); tensor names q, down, down_norm, up_k, up_v, o and gate (None:
-    no gate) relative to the prefix.
+    the layers' that read its rows; default: window); q_rank (None: queries are a projection of h); gate_kind; tensor names q,
+    down, down_norm, up_k, up_v, o, gate (None: no gate) and, with q_rank, q_down, q_down_norm relative to the prefix.
 
     32-bit: the latent's norm, the rotation, scores, softmax and its weights (the tensor-core kernels run in
     their variant whose weights keep 16 bits of mantissa), the gate. The stacked projection leaves 32-bit rows
@@ -50,11 +55,17 @@ class LatentAttention(Part):
         if self.row > ops.ATTENTION_SIMT_MAX_DIM:
             raise ValueError(f"latent_attention: kv_rank + rot_dim up to {ops.ATTENTION_SIMT_MAX_DIM} is supported, got {self.row}")
         self.gated = bool(p.get("gate"))
+        self.gate_kind = p.get("gate_kind", "channel")
+        if self.gate_kind not in ("channel", "head"):
+            raise ValueError(f"latent_attention: gate_kind is 'channel' or 'head', got {self.gate_kind!r}")
+        self.gate_rows = self.heads * (self.vdim if self.gate_kind == "channel" else 1) if self.gated else 0
+        self.q_rank = int(p.get("q_rank") or 0)
         self.window = int(p["window"]) if p.get("window") else None
         self.cache_window = int(p["cache_window"]) if p.get("cache_window") else self.window
         if self.window is not None and (self.window < 1 or self.cache_window < self.window):
             raise ValueError("latent_attention: a window holds at least the token itself, and the cached rows are kept at least that long")
         wanted = ["q", "up_k", "up_v", "o"] + (["gate"] if self.gated else []) + ([] if self.shares_cache else ["down", "down_norm"])
+        wanted += ["q_down", "q_down_norm"] if self.q_rank else []
         self.require(*wanted)
         self.names = {k: prefix + p[k] for k in wanted}
         self.position = build_part("position", p["position"], prefix)
@@ -64,13 +75,16 @@ class LatentAttention(Part):
 
     def tensor_specs(self):
         n = self.names
-        specs = [TensorSpec(n["q"], (self.heads * (self.dim + self.rot), self.hidden))]
+        specs = [TensorSpec(n["q"], (self.heads * (self.dim + self.rot), self.q_rank or self.hidden))]
+        if self.q_rank:
+            specs += [TensorSpec(n["q_down"], (self.q_rank, self.hidden)),
+                      TensorSpec(n["q_down_norm"], (self.q_rank,), kind="vector", init="ones")]
         if not self.shares_cache:
             specs += [TensorSpec(n["down"], (self.row, self.hidden)),
                       TensorSpec(n["down_norm"], (self.rank,), kind="vector", init="ones")]
         specs += [TensorSpec(n["up_k"], (self.heads * self.dim, self.rank)), TensorSpec(n["up_v"], (self.heads * self.vdim, self.rank))]
         if self.gated:
-            specs.append(TensorSpec(n["gate"], (self.heads * self.vdim, self.hidden)))
+            specs.append(TensorSpec(n["gate"], (self.gate_rows, self.hidden)))
         specs.append(TensorSpec(n["o"], (self.hidden, self.heads * self.vdim)))
         return specs + self.position.tensor_specs()
 
@@ -101,16 +115,21 @@ class LatentAttention(Part):
     def bind(self, tensors, runtime):
         super().bind(tensors, runtime)
         n = self.names
-        rows = [tensors.pop(n["q"])] + ([tensors.pop(n["gate"])] if self.gated else [])
+        # the stacked product's rows: [q, or the queries' latent | gate | latent and rotated key part (| padding)]
+        rows = [tensors.pop(n["q_down" if self.q_rank else "q"])]
+        self.gate_off = rows[0].shape[0]
+        self.w_up_q, self.q_down_norm = (tensors[n["q"]], tensors[n["q_down_norm"]]) if self.q_rank else (None, None)
+        if self.gated:
+            rows.append(tensors.pop(n["gate"]))
+        self.down_off = -1 if self.shares_cache else self.gate_off + self.gate_rows
+        self.down_norm = None
         if not self.shares_cache:
             rows.append(tensors.pop(n["down"]))
             self.down_norm = tensors[n["down_norm"]]
         used = sum(r.shape[0] for r in rows)
         if used % 16:           # whole 16-byte pieces per output row
             rows.append(torch.zeros((16 - used % 16, self.hidden), dtype=rows[0].dtype, device=rows[0].device))
-        self.w_in = torch.cat(rows, dim=0).contiguous()                    # [q | gate | down (| padding)]
-        self.q_off, self.gate_off = 0, self.heads * (self.dim + self.rot)
-        self.down_off = -1 if self.shares_cache else self.gate_off + (self.heads * self.vdim if self.gated else 0)
+        self.w_in = torch.cat(rows, dim=0).contiguous()
         # W_uk,h^T as the per-head product reads it: [heads, rank, dim]
         self.w_fold = tensors.pop(n["up_k"]).view(self.heads, self.dim, self.rank).transpose(1, 2).contiguous()
         self.w_up_v = tensors.pop(n["up_v"]).view(self.heads, self.vdim, self.rank).contiguous()
@@ -125,13 +144,19 @@ class LatentAttention(Part):
         tokens, group, room = h.shape[0], batch.groups[cache.group], self.room
         proj = self.runtime.linear(h, self.w_in, out_dtype=torch.float32)
         table = self.position.tables(batch)
+        q_rows, latent = proj, None
+        if self.q_rank:
+            latent = torch.empty((tokens, self.q_rank), dtype=h.dtype, device=h.device)
+        if latent is not None or not self.shares_cache:
+            ops.latent_rows(proj, self.down_off, self.down_norm, self.norm_eps, table, None if self.shares_cache else group.slot_map,
+                            None if self.shares_cache else cache.k_pool, self.rot, self.rank, cache.page_tokens,
+                            0, self.q_down_norm, latent)
+        if latent is not None:
+            q_rows = self.runtime.linear(latent, self.w_up_q, out_dtype=torch.float32)
+        # a head's query: its unrotated part through the key map, then its rotated part
         q = torch.empty((tokens, self.heads * room), dtype=h.dtype, device=h.device)
-        ops.latent_rows(proj, self.q_off, self.down_off, None if self.shares_cache else self.down_norm, self.norm_eps, table,
-                        None if self.shares_cache else group.slot_map, None if self.shares_cache else cache.k_pool, q,
-                        self.heads, self.dim, self.rot, self.rank, cache.page_tokens)
-        q3 = q.view(tokens, self.heads, room)
-        ops.heads_linear(proj[:, : self.heads * (self.dim + self.rot)].unflatten(1, (self.heads, self.dim + self.rot))[:, :, : self.dim],
-                         self.w_fold, q3[:, :, : self.rank])
+        ops.heads_linear(q_rows[:, : self.heads * (self.dim + self.rot)].unflatten(1, (self.heads, self.dim + self.rot)), self.w_fold,
+                         q.view(tokens, self.heads, room), tail=(table, self.rot))
         out = torch.empty((tokens, self.heads * room), dtype=h.dtype, device=h.device)
         if self.tensor_cores:
             ops.attention_bf16(q, cache, out, group.block_table, batch, self.heads, 1, room, cache.page_tokens, self.scale,
@@ -141,5 +166,5 @@ class LatentAttention(Part):
                               self.window or 0, room)
         gated = torch.empty((tokens, self.heads * self.vdim), dtype=h.dtype, device=h.device)
         ops.heads_linear(out.view(tokens, self.heads, room)[:, :, : self.rank], self.w_up_v, gated.view(tokens, self.heads, self.vdim),
-                         gate=proj[:, self.gate_off: self.gate_off + self.heads * self.vdim] if self.gated else None)
+                         gate=proj[:, self.gate_off: self.gate_off + self.gate_rows] if self.gated else None)
         return self.runtime.linear(gated, self.w_o)

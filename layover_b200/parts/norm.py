@@ -29,11 +29,22 @@ class Deferred:
     eps: float
 
 
+@dataclass
+class StreamUpdate:
+    """A sub-layer's output that has not joined the residual STREAMS yet (a model with several of them): all streams at
+    once from the old ones, x_t <- sum_s mix[s, t] x_s + gain[t] * value."""
+    value: torch.Tensor
+    mix: torch.Tensor       # float32 [streams, streams], [from, to]
+    gain: torch.Tensor      # float32 [streams]
+
+
 @register_norm("rmsnorm")
 class RMSNorm(Part):
     """y = weight * round(x * rsqrt(mean(x^2) + eps)), statistics in 32-bit (layover/model.py:25-36).
 
-    params: dim, eps, weight (tensor name relative to the prefix).
+    params: dim, eps, weight (tensor name relative to the prefix); optional weight_offset (default 0: added to the stored
+    weight in 32-bit when it is bound; 1 for weights that are stored around zero) and out_scale (default 1: a factor on y,
+    taken into the weight likewise).
     `forward(x, delta)` first adds `delta` into `x` (the residual sum, in 32-bit, rounded once)
     so that a block never launches a separate addition.
 
@@ -42,24 +53,42 @@ class RMSNorm(Part):
     returns: its output is normed, then added), and `extra` is one more 32-bit tensor to add (the
     embedding output, between the passes of layers that run several times). These take the
     32-bit-stream kernel, which rounds once, at the output; `add(x, delta, extra)` is the same
-    without a norm of the sum."""
+    without a norm of the sum.
+
+    Over several residual streams (x [T, streams, dim]) `read_streams` norms a weighted sum of them, after the pending
+    `StreamUpdate` has joined, in one kernel; `forward` of such a stream is the norm of their plain sum."""
 
     def __init__(self, params, prefix):
         super().__init__(params, prefix)
         self.require("dim", "eps", "weight")
         self.dim, self.eps = int(params["dim"]), float(params["eps"])
         self.weight_name = prefix + params["weight"]
+        self.weight_offset, self.out_scale = float(params.get("weight_offset", 0.0)), float(params.get("out_scale", 1.0))
         self.weight = None
 
     def tensor_specs(self):
-        return [TensorSpec(self.weight_name, (self.dim,), kind="vector", init="ones")]
+        return [TensorSpec(self.weight_name, (self.dim,), kind="vector", init="ones", init_offset=-self.weight_offset)]
 
     def bind(self, tensors, runtime):
         super().bind(tensors, runtime)
         self.weight = tensors[self.weight_name]
+        if self.weight_offset != 0.0 or self.out_scale != 1.0:
+            self.weight = (self.weight + self.weight_offset) * self.out_scale
 
     def kernel_libraries(self, dtype):
         return ("elementwise",)
+
+    def read_streams(self, x: torch.Tensor, pending: StreamUpdate | None, read: torch.Tensor | None, rows=None, shift=None):
+        """(streams, h): x [T, streams, dim] with `pending` joined, and the norm of its sum weighted by `read` [streams]
+        (None: the plain sum). The streams come in another buffer; with nothing pending they are x itself, with `rows` (only
+        those rows of h) nobody needs them: None. `shift` = (mu, state, batch): h moves towards the h of the token before it
+        by the share mu of each channel (see `ops.stream_norm`)."""
+        n = x.shape[0] if rows is None else rows.shape[0]
+        out = torch.empty((n, self.dim), dtype=self.runtime.dtype, device=x.device)
+        update = None if pending is None else (pending.value, pending.mix, pending.gain)
+        made = torch.empty(x.shape, dtype=torch.float32, device=x.device) if update is not None and rows is None else None
+        ops.stream_norm(x, update, read, self.weight, self.eps, out, made, rows, shift)
+        return (made if made is not None else (x if rows is None else None)), out
 
     def defer(self, value: torch.Tensor) -> Deferred:
         """`value` as something this norm is to be applied to when it is added to the stream."""
@@ -67,6 +96,10 @@ class RMSNorm(Part):
 
     def forward(self, x: torch.Tensor, delta, rows: torch.Tensor | None = None,
                 extra: torch.Tensor | None = None) -> torch.Tensor:
+        if x.dim() == 3:        # several streams: the norm of their sum
+            if extra is not None:
+                raise ValueError("a norm of several streams takes no extra summand")
+            return self.read_streams(x, delta, None, rows)[1]
         n = x.shape[0] if rows is None else rows.shape[0]
         wide = x.dtype == torch.float32 and self.runtime.dtype != torch.float32
         if not (wide or isinstance(delta, Deferred) or extra is not None):

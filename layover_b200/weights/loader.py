@@ -32,7 +32,8 @@ class TensorSpec:
     name: str
     shape: tuple[int, ...]
     kind: str = "matrix"
-    init: str = "normal"          # "normal": N(0, std); "ones": 1 + N(0, norm_std); "zeros"
+    init: str = "normal"          # "normal": N(0, std); "ones": 1 + N(0, norm_std); "zeros"; "eye": "ones" on the diagonal, N(0, norm_std) off it
+    init_offset: float = 0.0      # added to what `init` gives (weights stored around zero where their use adds the one)
     optional_alias: str | None = None  # stored name that may stand in (a tied head reads the embedding)
 
     def __post_init__(self):

@@ -4,7 +4,8 @@ The reference has no such mode; its tests seed torch and take the layers' defaul
 initialisation (tests/test_hot_path.py:23-26). Here every tensor is drawn from its own
 generator, seeded by the run's seed and the tensor's name, so a tensor's values do not depend
 on which other tensors exist or in which order they are made: matrices ~ N(0, std), norm
-weights 1 + N(0, norm_std).
+weights 1 + N(0, norm_std) (around zero where the model stores them so), mixing matrices of
+residual streams the identity + N(0, norm_std).
 """
 
 from __future__ import annotations
@@ -34,7 +35,9 @@ def random_tensor(spec: TensorSpec, seed: int, std: float, norm_std: float, devi
         return torch.zeros(spec.shape, dtype=torch.float32, device=device)
     noise = torch.randn(spec.shape, generator=gen, dtype=torch.float32, device=device)
     if spec.init == "ones":
-        return 1.0 + norm_std * noise
+        return 1.0 + norm_std * noise + spec.init_offset
+    if spec.init == "eye":
+        return torch.eye(*spec.shape, device=device) + norm_std * noise
     return std * noise
 
 
