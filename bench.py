@@ -1,7 +1,7 @@
 """Decode and prefill throughput of the engine on one B200, random weights of a named Qwen3 shape.
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--impl ours|reference]
-                    [--config 4b|4b-fp32|8b-mixed|32b-long|topidra|limazen|kirenex|vopozen|fimilix]
+                    [--config 4b|4b-fp32|8b-mixed|32b-long|topidra|limazen|kirenex|vopozen|fimilix|mimitar]
 
 A step is one decode step. Every run prints ONE JSON line on standard output.
 
@@ -62,6 +62,13 @@ around attention alone) and Kirenex (a recurrence beside the attention in every 
 active width) at equal width and heads, four layers each: prefill of 2,048 tokens and decode at batch 8 for all
 three, then Fimilix's own kernels alone with the like kernels of the other paths (`--only kernels`: those alone).
 
+--config mimitar: the Mimitar design (two residual streams mixed anew around every sub-layer, a token shift ahead of
+every mixer; attention with whole-row norms and capped scores, latent attention with latent queries, dense and routed
+feed-forwards with clipped gates) beside Vopozen, the closest design the engine has (attention and latent attention over
+one 32-bit stream, dense and routed feed-forwards), with the same kinds of layers at equal width, heads, head sizes and
+weights, four layers each: prefill of 2,048 tokens and decode at batch 8 for both, then Mimitar's own kernels alone with
+the like kernels of the other paths (`--only kernels`: those alone).
+
 Peaks come from MEASURED_PEAKS.json beside this file when it exists (else 6.65 TB/s and
 1.59 PFLOP/s, an earlier measurement of the same kind of GPU). Inputs are synthetic token ids;
 weights are seeded random values of the named shape. Weights (8 GB and more) are larger than the
@@ -91,7 +98,7 @@ FALLBACK_PEAKS = {"hbm_gbs": 6650.0, "bf16_tflops": 1590.0, "bf16_tflops_sustain
 FP32_TFLOPS = 75.0       # nominal FFMA rate of the part; only the 32-bit path's prefill fraction uses it
 CONFIGS = {"4b": ("qwen3-4b", "bf16"), "4b-fp32": ("qwen3-4b", "fp32"), "8b-mixed": ("qwen3-8b", "bf16"),
            "32b-long": ("qwen3-32b", "bf16"), "topidra": ("topidra", "bf16"), "limazen": ("limazen", "bf16"), "kirenex": ("kirenex", "bf16"), "vopozen": ("vopozen", "bf16"),
-           "fimilix": ("fimilix", "bf16")}
+           "fimilix": ("fimilix", "bf16"), "mimitar": ("mimitar", "bf16")}
 METRIC = "decode tokens/s (Qwen3-4B shape, batch 8, context 2048->4096)"
 
 
@@ -1183,9 +1190,8 @@ def kirenex_kernels(pk: dict) -> dict:
         q = torch.zeros(tokens, l_heads * room, device=dev, dtype=bf)
         wn = torch.ones(rank, device=dev)
         gate_off = l_heads * (dim + rot)
-        point(f"latent_rows_{tokens}", lambda i: ops.latent_rows(proj[i % ROT], 0, gate_off + l_heads * dim, wn, 1e-6, half, slots, pool, q,
-                                                               l_heads, dim, rot, rank, page), ROT,
-              nbytes=tokens * ((l_heads * rot + row) * 4 + (l_heads * rot + room) * 2))
+        point(f"latent_rows_{tokens}", lambda i: ops.latent_rows(proj[i % ROT], gate_off + l_heads * dim, wn, 1e-6, half, slots, pool, rot, rank,
+                                                               page), ROT, nbytes=tokens * (row * 4 + room * 2))
         w_fold = [torch.randn(l_heads, rank, dim, device=dev, dtype=bf) * 0.05 for _ in range(2)]
         w_up = [torch.randn(l_heads, dim, rank, device=dev, dtype=bf) * 0.05 for _ in range(2)]
         q3 = q.view(tokens, l_heads, room)
@@ -1193,9 +1199,9 @@ def kirenex_kernels(pk: dict) -> dict:
         gated = torch.empty(tokens, l_heads, dim, device=dev, dtype=bf)
         weight_bytes = l_heads * rank * dim * 2
         point(f"heads_linear_fold_{tokens}",
-              lambda i: ops.heads_linear(proj[i % ROT][:, :gate_off].unflatten(1, (l_heads, dim + rot))[:, :, :dim], w_fold[i % 2],
-                                         q3[:, :, :rank]), ROT,
-              nbytes=weight_bytes + tokens * l_heads * (dim * 4 + rank * 2), flops=2.0 * tokens * l_heads * dim * rank,
+              lambda i: ops.heads_linear(proj[i % ROT][:, :gate_off].unflatten(1, (l_heads, dim + rot)), w_fold[i % 2], q3,
+                                         tail=(half, rot)), ROT,
+              nbytes=weight_bytes + tokens * l_heads * ((dim + rot) * 4 + room * 2), flops=2.0 * tokens * l_heads * dim * rank,
               peak_flops=FP32_TFLOPS * 1e12)
         point(f"heads_linear_values_gate_{tokens}",
               lambda i: ops.heads_linear(heads_out[:, :, :rank], w_up[i % 2], gated, gate=proj[i % ROT][:, gate_off: gate_off + l_heads * dim]),
@@ -1935,6 +1941,265 @@ def run_fimilix(args, pk, pk_source) -> dict:
             "sizes": sizes, "kernels": fimilix_kernels(pk)}
 
 
+# --------------------------------------------------------------------------------------- Mimitar beside Vopozen
+MIMITAR_SIZES = {   # name: (width, heads, KV heads, head size, dense width, latents of keys and of queries, experts, chosen, expert and shared width)
+    "1024": (1024, 8, 4, 128, 3072, 192, 384, 16, 4, 768, 1024),
+    "2048": (2048, 16, 8, 128, 6144, 192, 768, 32, 4, 1536, 2048),
+    "4096": (4096, 32, 8, 128, 12288, 192, 1536, 32, 4, 3072, 4096)}
+MIMITAR_LAYERS, MIMITAR_VOCAB, MIMITAR_ROT, MIMITAR_STREAMS, MIMITAR_SPAN, MIMITAR_CAP = 4, 32768, 64, 2, 8192, 40.0
+MIMITAR_GROUPS, MIMITAR_KEEP = 4, 2
+
+
+def mimitar_pair(size: str):
+    """(Mimitar, Vopozen) configurations of equal width, heads, head size, latent, feed-forward and depth: attention and
+    latent attention over a dense feed-forward, then both over routed experts with a shared one. Vopozen's experts have no
+    gate and are half as wide again, so that both read the same bytes; its chunk and window are longer than any request here,
+    so that both attend over every earlier token."""
+    import layover_b200 as lb
+    from layover_b200.config.mimitar import capped_layer, dense_mlp, latent_layer, routed_mlp
+    from layover_b200.config.vopozen import chunked_layer, windowed_latent_layer
+
+    width, heads, kv, dim, ff, rank, q_rank, experts, top, expert_ff, shared_ff = MIMITAR_SIZES[size]
+    routed = routed_mlp(experts, top, expert_ff, 7.0, (MIMITAR_GROUPS, MIMITAR_KEEP), (shared_ff, 7.0))
+
+    def attention(mlp):
+        return capped_layer(heads, kv, dim, dim, 500000.0, dim // 2, bands=(8.0, 1.0, 4.0, 4096), softcap=MIMITAR_CAP, mlp=mlp)
+
+    def latent(mlp):
+        return latent_layer(heads, dim, MIMITAR_ROT, dim, rank, q_rank, 10000.0, ramp=(4.0, 4096, 32.0, 1.0), mlp=mlp)
+    mimitar = lb.MimitarConfig(vocab=MIMITAR_VOCAB, width=width, streams=MIMITAR_STREAMS, residual_mult=0.5, logit_scale=0.5,
+                               layers=(attention(dense_mlp(ff)), latent(dense_mlp(ff)), attention(routed), latent(routed)))
+    other = dict(experts=experts, top=top, expert_ff=expert_ff * 3 // 2, shared_ff=shared_ff, groups=MIMITAR_GROUPS, keep=MIMITAR_KEEP)
+    chunked = dict(rot_dims=dim // 2, base=1000000.0)
+    vopozen = lb.VopozenConfig(vocab=MIMITAR_VOCAB, width=width, residual_mult=0.8, layers=(
+        chunked_layer(heads, kv, dim, MIMITAR_SPAN, ff=ff, **chunked),
+        windowed_latent_layer(heads, dim, MIMITAR_ROT, dim, rank, MIMITAR_SPAN, base=10000.0, ff=ff),
+        chunked_layer(heads, kv, dim, MIMITAR_SPAN, **chunked, **other),
+        windowed_latent_layer(heads, dim, MIMITAR_ROT, dim, rank, MIMITAR_SPAN, base=10000.0, **other)))
+    return mimitar, vopozen
+
+
+def mimitar_kernels(pk: dict) -> dict:
+    """Mimitar's own kernels alone at the 2048 layer size, each with the like kernel of the other paths: microseconds
+    (kernels back to back in a replayed graph, operands rotating through more memory than the L2 holds) and the fraction
+    of the measured peak that bounds it."""
+    import types
+    import torch
+    from layover_b200 import ops
+
+    width, heads, kv, dim, ff, rank, q_rank, experts, top, expert_ff, shared_ff = MIMITAR_SIZES["2048"]
+    S, rot = MIMITAR_STREAMS, MIMITAR_ROT
+    dev, bf = "cuda", torch.bfloat16
+    hbm, tensor = pk["hbm_gbs"] * 1e9, pk["bf16_tflops"] * 1e12
+    out = {}
+
+    def point(name, fn, calls, nbytes=None, flops=None, peak_flops=None):
+        us = graph_time(fn, calls) * 1000.0
+        row = {"us": round(us, 2)}
+        if nbytes:
+            row["of_hbm"] = round(nbytes / (us * 1e-6) / hbm, 3)
+        if flops:
+            row["of_flops"] = round(flops / (us * 1e-6) / (peak_flops or tensor), 3)
+        out[name] = row
+
+    ROT, page = 8, PAGE
+    n = heads * dim
+    own, mixer = ops.stream_shift_tokens(), ops.wkv_mix_tokens()
+
+    # ---- the streams between two sub-layers, without and with a token shift; beside one stream's add + norm and the shift alone
+    for tokens, seqs in ((2048, 1), (8, 8), (64, 64)):
+        per = tokens // seqs
+        tag = "prompt2048" if seqs == 1 else f"decode_b{seqs}"
+        R = ROT if tokens > 64 else 256             # as many buffers as fill the L2 and more, whatever the step
+
+        def tiles_of(size):
+            listed = [(s, q0) for s in range(seqs) for q0 in range(0, per, size)]
+            return types.SimpleNamespace(tile_seq=torch.tensor([t[0] for t in listed], dtype=torch.int32, device=dev),
+                                         tile_q0=torch.tensor([t[1] for t in listed], dtype=torch.int32, device=dev), count=len(listed))
+        batch = types.SimpleNamespace(cu_q=torch.arange(0, tokens + 1, per, dtype=torch.int32, device=dev), n_seqs=seqs, n_tokens=tokens,
+                                      state_slots=torch.arange(seqs, dtype=torch.int32, device=dev), tiles={own: tiles_of(own), mixer: tiles_of(mixer)})
+        x = [torch.randn(tokens, S, width, device=dev) for _ in range(R)]
+        y = [torch.randn(tokens, width, device=dev, dtype=bf) for _ in range(R)]
+        w, mu, read = torch.ones(width, device=dev), torch.rand(width, device=dev), torch.rand(S, device=dev)
+        update = (torch.eye(S, device=dev) + 0.1, torch.rand(S, device=dev))
+        o = torch.empty(tokens, width, device=dev, dtype=bf)
+        made = [torch.empty_like(x[0]) for _ in range(R)]
+        state = torch.zeros(R, seqs + 1, width, device=dev)
+        point(f"stream_norm_{tag}", lambda i: ops.stream_norm(x[i % R], (y[i % R], *update), read, w, 1e-6, o, made[i % R]), R,
+              nbytes=tokens * width * (2 * S * 4 + 2 + 2))
+        point(f"stream_norm_shift_{tag}", lambda i: ops.stream_norm(x[i % R], (y[i % R], *update), read, w, 1e-6, o, made[i % R],
+                                                                   shift=(mu, state[i % R], batch)), R,
+              nbytes=tokens * width * (2 * S * 4 + 2 + 2) + 2 * seqs * width * 4)
+        one = [t.view(tokens * S, width)[:tokens] for t in x]
+        point(f"like:residual_rmsnorm_{tag}", lambda i: ops.residual_rmsnorm(one[i % R], y[i % R], None, 0.0, None, w, 1e-6, o), R,
+              nbytes=tokens * width * (4 + 4 + 2 + 2))
+        mixes, mus = torch.empty(1, tokens, width, device=dev, dtype=bf), mu[None].contiguous()
+        point(f"like:wkv_shift_mix_one_{tag}", lambda i: ops.wkv_shift_mix(y[i % R], mus, state[i % R], 0, batch, mixes), R,
+              nbytes=tokens * width * (2 + 2))
+        if seqs == 1:
+            rows = torch.tensor([tokens - 1], dtype=torch.int32, device=dev)
+            last = torch.empty(1, width, device=dev, dtype=bf)
+            point("stream_norm_last_row", lambda i: ops.stream_norm(x[i % R], (y[i % R], *update), None, w, 1e-6, last, rows=rows), R)
+            point("like:residual_rmsnorm_last_row", lambda i: ops.residual_rmsnorm(one[i % R], y[i % R], None, 0.0, None, w, 1e-6, last, rows), R)
+        del x, y, made, one
+        torch.cuda.empty_cache()
+
+    ROT = 6
+    for tokens in (2048, 8):
+        # ---- q and k normed over whole rows, rotation of half a head, page write; beside the same kernel with a norm per head
+        pos = torch.arange(tokens, dtype=torch.int32, device=dev)
+        half = torch.empty(tokens, 2, dim // 4, device=dev)
+        ops.rope_table(pos, torch.rand(dim // 4, device=dev), half)
+        slots = torch.arange(tokens, dtype=torch.int32, device=dev)
+        pool = torch.zeros(2, tokens // page + 2, kv, page, dim, device=dev, dtype=bf)
+        qo = torch.empty(tokens, n, device=dev, dtype=bf)
+        rows_n = (heads + 2 * kv) * dim
+        proj = [torch.randn(tokens, rows_n, device=dev) for _ in range(ROT)]
+        for name, whole, wq, wk in (("heads_whole_norm_rope_kv", True, torch.ones(n, device=dev), torch.ones(kv * dim, device=dev)),
+                                    ("like:heads_norm_rope_kv", False, torch.ones(dim, device=dev), torch.ones(dim, device=dev))):
+            point(f"{name}_{tokens}",
+                  lambda i: ops.heads_bias_rope_kv(proj[i % ROT], qo, pool[0], pool[1], None, None, None, half, slots, None, 0, None, heads, kv, dim,
+                                                   dim, page, wq, wk, 1e-6, whole_norm=whole), ROT, nbytes=tokens * rows_n * (4 + 2))
+        del proj
+        # ---- the latents' norms and page write; the queries' product; the key map with the rotated tail; values with a gate
+        row, room = rank + rot, -(-(rank + rot) // 16) * 16
+        n_proj = q_rank + heads * dim + row
+        n_proj += -n_proj % 16
+        proj = [torch.randn(tokens, n_proj, device=dev) for _ in range(ROT)]
+        lpool = torch.zeros(tokens // page + 2, 1, page, room, device=dev, dtype=bf)
+        table = torch.empty(tokens, 2, rot // 2, device=dev)
+        ops.rope_table(pos, torch.rand(rot // 2, device=dev), table)
+        wn, wqn = torch.ones(rank, device=dev), torch.ones(q_rank, device=dev)
+        cq = torch.empty(tokens, q_rank, device=dev, dtype=bf)
+        down = q_rank + heads * dim
+        point(f"latent_rows_both_{tokens}", lambda i: ops.latent_rows(proj[i % ROT], down, wn, 1e-6, table, slots, lpool, rot, rank, page, 0, wqn, cq),
+              ROT, nbytes=tokens * ((row + q_rank) * 4 + (room + q_rank) * 2))
+        point(f"like:latent_rows_{tokens}", lambda i: ops.latent_rows(proj[i % ROT], down, wn, 1e-6, table, slots, lpool, rot, rank, page), ROT,
+              nbytes=tokens * (row * 4 + room * 2))
+        w_uq = [torch.randn(heads * (dim + rot), q_rank, device=dev, dtype=bf) * 0.05 for _ in range(16)]
+        w_q = [torch.randn(heads * (dim + rot), width, device=dev, dtype=bf) * 0.05 for _ in range(16)]
+        h = torch.randn(tokens, width, device=dev, dtype=bf)
+        q_rows = torch.empty(tokens, heads * (dim + rot), device=dev)
+        point(f"latent_queries_product_{tokens}", lambda i: ops.gemm_bf16(cq, w_uq[i % 16], q_rows), 16,
+              nbytes=heads * (dim + rot) * q_rank * 2 + tokens * (q_rank * 2 + heads * (dim + rot) * 4), flops=2.0 * tokens * heads * (dim + rot) * q_rank)
+        point(f"like:queries_product_{tokens}", lambda i: ops.gemm_bf16(h, w_q[i % 16], q_rows), 16,
+              nbytes=heads * (dim + rot) * width * 2 + tokens * (width * 2 + heads * (dim + rot) * 4), flops=2.0 * tokens * heads * (dim + rot) * width)
+        w_fold = [torch.randn(heads, rank, dim, device=dev, dtype=bf) * 0.05 for _ in range(2)]
+        w_up = [torch.randn(heads, dim, rank, device=dev, dtype=bf) * 0.05 for _ in range(2)]
+        q = torch.zeros(tokens, heads, room, device=dev, dtype=bf)
+        q_in = q_rows.unflatten(1, (heads, dim + rot))
+        cost = dict(flops=2.0 * tokens * heads * dim * rank, peak_flops=FP32_TFLOPS * 1e12)
+        weight_bytes = heads * rank * dim * 2
+        point(f"heads_linear_fold_and_tail_{tokens}", lambda i: ops.heads_linear(q_in, w_fold[i % 2], q, tail=(table, rot)), ROT,
+              nbytes=weight_bytes + tokens * heads * ((dim + rot) * 4 + room * 2), **cost)
+        point(f"like:heads_linear_fold_{tokens}", lambda i: ops.heads_linear(q_in[:, :, :dim], w_fold[i % 2], q[:, :, :rank]), ROT,
+              nbytes=weight_bytes + tokens * heads * (dim * 4 + rank * 2), **cost)
+        gated = torch.empty(tokens, heads, dim, device=dev, dtype=bf)
+        for name, at in (("heads_linear_values_head_gate", heads), ("like:heads_linear_values_channel_gate", heads * dim)):
+            point(f"{name}_{tokens}", lambda i: ops.heads_linear(q[:, :, :rank], w_up[i % 2], gated, gate=proj[i % ROT][:, q_rank: q_rank + at]), ROT,
+                  nbytes=weight_bytes + tokens * heads * (rank * 2 + dim * 2) + tokens * at * 4, **cost)
+        del proj, w_uq, w_q
+        # ---- the dense feed-forward's first product with the clipped gate in its epilogue; beside silu
+        wide = [torch.randn(2 * ff, width, device=dev, dtype=bf) * 0.02 for _ in range(4)]
+        act = torch.empty(tokens, ff, device=dev, dtype=bf)
+        cost = dict(nbytes=2 * ff * width * 2, flops=2.0 * tokens * 2 * ff * width)
+        point(f"gate_up_clipped_{tokens}", lambda i: ops.gemm_tcgen05(h, wide[i % 4], act, epilogue="clipped_swiglu", limit=7.0, slope=1.702), 4, **cost)
+        point(f"like:gate_up_swiglu_{tokens}", lambda i: ops.gemm_tcgen05(h, wide[i % 4], act, epilogue="swiglu"), 4, **cost)
+        both = torch.empty(tokens, 2 * ff, device=dev, dtype=bf)
+
+        def product_then_gate(i):
+            ops.gemm_tcgen05(h, wide[i % 4], both)
+            ops.gated_act(both, act, "clipped_swiglu", block=ops.SWIGLU_BLOCK, limit=7.0, slope=1.702)
+        point(f"like:gate_up_then_clipped_gate_{tokens}", product_then_gate, 4, **cost)
+        del wide, both
+        # ---- the router: softmax over all experts, the groups of the best; beside corrected sigmoids and groups of two
+        hs = [torch.randn(tokens, width, device=dev, dtype=bf) for _ in range(ROT)]
+        router = torch.randn(experts, width, device=dev) * 0.05
+        ids, scores = torch.empty(tokens, top, dtype=torch.int32, device=dev), torch.empty(tokens, top, device=dev)
+        groups = dict(groups=MIMITAR_GROUPS, keep_groups=MIMITAR_KEEP, renormalize=True)
+        kinds = (("softmax_all_groups", dict(groups, score="softmax_all", group_score="best")),
+                 ("like:sigmoid_corrected_groups", dict(groups, correction=torch.randn(experts, device=dev))))
+        matrix = torch.zeros(-(-experts // 8) * 8, width, device=dev, dtype=bf)
+        matrix[:experts] = router.to(bf)
+        logits = torch.empty(tokens, matrix.shape[0], device=dev)
+
+        def route_product(i, options):
+            ops.gemm_tcgen05(hs[i % ROT], matrix, logits)
+            ops.moe_select(logits, experts, top, ids, scores, **options)
+        for name, options in kinds:
+            prefix, _, kind = name.rpartition(":")
+            prefix += ":" if prefix else ""
+            if tokens > 64:
+                point(f"{prefix}moe_route_product_{kind}_{tokens}", lambda i: route_product(i, options), ROT, nbytes=tokens * width * 2 + experts * width * 2)
+            else:
+                point(f"{prefix}moe_route_{kind}_{tokens}", lambda i: ops.moe_route(hs[i % ROT], router, top, ids, scores, **options), ROT,
+                      nbytes=tokens * width * 2 + experts * width * 4)
+        del hs
+
+    # ---- attention with capped scores beside none, latent attention (the same kernels as Kirenex's and Vopozen's)
+    sms = ops.gemm_scratch(torch.device(dev))[2]
+    row, room = rank + rot, -(-(rank + rot) // 16) * 16
+    for tokens, seqs, ctx in ((2048, 1, 2048), (8, 8, 3072), (64, 64, 3072)):
+        pages_per, R, per = -(-ctx // page), ROT if seqs < 64 else 2, tokens // seqs
+        table = torch.arange(seqs * pages_per, dtype=torch.int32, device=dev).view(seqs, pages_per)
+        cu = torch.arange(0, tokens + 1, per, dtype=torch.int32, device=dev)
+        lens = torch.full((seqs,), ctx, dtype=torch.int32, device=dev)
+        pools = [torch.randn(2, seqs * pages_per + 1, kv, page, dim, device=dev, dtype=bf) for _ in range(R)]
+        lpools = [torch.randn(seqs * pages_per + 1, 1, page, room, device=dev, dtype=bf) for _ in range(R)]
+        q, lq = torch.randn(tokens, n, device=dev, dtype=bf), torch.randn(tokens, heads * room, device=dev, dtype=bf)
+        o, lo = torch.empty_like(q), torch.empty_like(lq)
+        if per > 1:
+            bq = ops.attention_mma_block_queries()
+            tq = torch.arange(0, per, bq, dtype=torch.int32, device=dev)
+            ts, pairs = torch.zeros_like(tq), per * (per + 1) // 2
+            for name, cap in (("capped_attention", MIMITAR_CAP), ("like:exact_attention", 0.0)):
+                point(f"{name}_prompt2048",
+                      lambda i: ops.attention_prefill_bf16(q, pools[i % R][0], pools[i % R][1], o, table, cu, lens, ts, tq, tq.numel(), heads, kv, dim,
+                                                           page, dim ** -0.5, 0, exact_weights=True, softcap=cap), R, flops=4.0 * heads * dim * 1.25 * pairs)
+            point("latent_attention_prompt2048",
+                  lambda i: ops.attention_prefill_bf16(lq, lpools[i % R], lpools[i % R], lo, table, cu, lens, ts, tq, tq.numel(), heads, 1, room, page,
+                                                       row ** -0.5, 0, exact_weights=True), R, flops=2.0 * heads * room * 2.5 * pairs)
+        else:
+            splits, stages = ops.decode_plan(seqs, heads, kv, dim, ctx, sms)
+            for name, cap in (("capped_attention", MIMITAR_CAP), ("like:exact_attention", 0.0)):
+                point(f"{name}_decode_b{seqs}",
+                      lambda i: ops.attention_decode_bf16(q, pools[i % R][0], pools[i % R][1], o, table, cu, lens, None, seqs, heads, kv, dim, page,
+                                                          dim ** -0.5, 0, splits, stages, exact_weights=True, softcap=cap), R,
+                      nbytes=seqs * kv * ctx * 2 * dim * 2)
+            splits, stages = ops.decode_plan(seqs, heads, 1, room, ctx, sms)
+            point(f"latent_attention_decode_b{seqs}",
+                  lambda i: ops.attention_decode_bf16(lq, lpools[i % R], lpools[i % R], lo, table, cu, lens, None, seqs, heads, 1, room, page,
+                                                      row ** -0.5, 0, splits, stages, exact_weights=True), R, nbytes=seqs * ctx * room * 2)
+        del pools, lpools
+        torch.cuda.empty_cache()
+    return out
+
+
+def run_mimitar(args, pk, pk_source) -> dict:
+    import torch
+    import layover_b200 as lb
+
+    gen = torch.Generator().manual_seed(0)
+    sizes = {}
+    for size in MIMITAR_SIZES if args.only != "kernels" else ():
+        row = {}
+        for name, cfg in zip(("mimitar", "vopozen"), mimitar_pair(size)):
+            model = lb.random_model(cfg, seed=0, device="cuda", dtype=args.dtype, std=0.02)
+            prefill = prefill_point(model, gen, repeats=5)
+            decode = decode_point(model, args.batch, min(args.steps, 64), args.warmup, gen)
+            row[name] = {"prefill_tok_s": round(prefill["tok_s"], 1), "prefill_ms": round(prefill["ms"], 3),
+                         "decode_tok_s": round(decode["tok_s"], 1), "decode_ms_per_step": round(decode["ms_per_step"], 4),
+                         "launches_per_step": round(decode["launches"] / min(args.steps, 64), 1),
+                         "weight_gb": round(model.weight_bytes() / 1e9, 3)}
+            del model
+            torch.cuda.empty_cache()
+        sizes[size] = row
+    return {"metric": "Mimitar beside Vopozen with the same kinds of layers at equal width, heads and weights: prefill of 2,048 tokens "
+                      f"and decode at batch {args.batch}, {MIMITAR_LAYERS} layers, vocabulary {MIMITAR_VOCAB}",
+            "dtype": args.dtype, "data": "synthetic token ids, seeded random weights", "peaks": pk_source,
+            "streams": MIMITAR_STREAMS, "sizes": sizes, "kernels": mimitar_kernels(pk)}
+
+
 def lb_preset(name: str):
     import layover_b200 as lb
     return lb.preset(name)
@@ -1961,6 +2226,8 @@ def run_ours(args) -> dict:
         return run_vopozen(args, pk, pk_source)
     if args.config == "fimilix":
         return run_fimilix(args, pk, pk_source)
+    if args.config == "mimitar":
+        return run_mimitar(args, pk, pk_source)
     if args.only == "kernels":
         return {"only": "kernels", **kernel_points(args.model, pk, with_library=True)}
     if args.only == "plans":
@@ -2107,7 +2374,7 @@ def main(argv=None) -> int:
     parser.add_argument("--config", default="4b", choices=sorted(CONFIGS),
                         help="4b: the headline; 4b-fp32: the 32-bit path; 8b-mixed: 32 mixed requests through the "
                              "scheduler; 32b-long: 8 x 32,768-token contexts; topidra / limazen: that design beside "
-                             "Qwen3 at equal layer sizes, and its kernels alone; kirenex: that design beside Topidra; vopozen: that design beside Kirenex; fimilix: that design beside Limazen and Kirenex")
+                             "Qwen3 at equal layer sizes, and its kernels alone; kirenex: that design beside Topidra; vopozen: that design beside Kirenex; fimilix: that design beside Limazen and Kirenex; mimitar: that design beside Vopozen")
     parser.add_argument("--model", default=None, help="a preset's name instead of the one --config names")
     parser.add_argument("--dtype", default=None, choices=["bf16", "fp32"])
     parser.add_argument("--batch", type=int, default=8)
