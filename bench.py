@@ -2004,7 +2004,7 @@ def mimitar_kernels(pk: dict) -> dict:
 
     ROT, page = 8, PAGE
     n = heads * dim
-    own, mixer = ops.stream_shift_tokens(), ops.wkv_mix_tokens()
+    mixer = ops.wkv_mix_tokens()
 
     # ---- the streams between two sub-layers, without and with a token shift; beside one stream's add + norm and the shift alone
     for tokens, seqs in ((2048, 1), (8, 8), (64, 64)):
@@ -2017,7 +2017,7 @@ def mimitar_kernels(pk: dict) -> dict:
             return types.SimpleNamespace(tile_seq=torch.tensor([t[0] for t in listed], dtype=torch.int32, device=dev),
                                          tile_q0=torch.tensor([t[1] for t in listed], dtype=torch.int32, device=dev), count=len(listed))
         batch = types.SimpleNamespace(cu_q=torch.arange(0, tokens + 1, per, dtype=torch.int32, device=dev), n_seqs=seqs, n_tokens=tokens,
-                                      state_slots=torch.arange(seqs, dtype=torch.int32, device=dev), tiles={own: tiles_of(own), mixer: tiles_of(mixer)})
+                                      state_slots=torch.arange(seqs, dtype=torch.int32, device=dev), tiles={mixer: tiles_of(mixer)})
         x = [torch.randn(tokens, S, width, device=dev) for _ in range(R)]
         y = [torch.randn(tokens, width, device=dev, dtype=bf) for _ in range(R)]
         w, mu, read = torch.ones(width, device=dev), torch.rand(width, device=dev), torch.rand(S, device=dev)

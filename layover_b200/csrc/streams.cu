@@ -10,11 +10,11 @@
 // first token the request's state row. Everything is 32-bit arithmetic in a fixed order, rounded once at the store.
 //
 // The streams are written to another buffer than they are read from (x_out null: not written at all), which is what lets
-// blocks compute a neighbour's h again instead of waiting for it: a block of the shifted form owns SHIFT_TOKENS tokens of
-// one sequence and first computes the h of the token before them. The block with a sequence's first token of the step
-// reads the state row and, at the end, writes it: with its own last token's h, or, where the sequence goes on in other
-// blocks, with the last token's h computed once more. So a row of state has one reader and writer, whatever the cut,
-// and the value has the bits that any other block would have given it.
+// blocks compute a neighbour's h again instead of waiting for it: a block of the shifted form owns one token and computes
+// the h of the token before it as well (the reads are the neighbour's, a moment apart: the L2 serves one of the two). The
+// block with a sequence's first token of the step reads the state row and, at the end, writes it: with its own h, or, where
+// the sequence goes on in other blocks, with the last token's h computed once more. So a row of state has one reader and
+// writer, whatever the cut, and the value has the bits that any other block would have given it.
 //
 // `x_stream` is the distance between a token's streams; 0 lets one row stand for all of them (they start out equal).
 #include <math.h>
@@ -22,7 +22,6 @@
 #include "common.cuh"
 
 namespace {
-constexpr int SHIFT_TOKENS = 4;
 constexpr int MAX_STREAMS = 16;
 constexpr int MAX_THREADS = 512;      // so widths up to 8192 (4096 where they are no multiple of 4)
 
@@ -67,11 +66,11 @@ struct StreamProblem {
   int width, streams;
 };
 
-// One token by all threads of the block: thread i owns channel pieces i, i + blockDim, ... (NP of them at most) and gets
-// its channels of h. S: the number of streams, 0 for any number (then x is read once per stream that is made).
+// One token by all threads of the block: thread i owns channel pieces i, i + blockDim, ... (NP of them at most), gets its
+// channels of u and returns their sum of squares. S: the number of streams, 0 for any number (then x is read once per
+// stream that is made).
 template <typename T, int S, int C, int NP>
-__device__ __forceinline__ void token_norm(const StreamProblem& p, const float* small, size_t token, bool write, float* scratch,
-                                           float (&h)[NP][C]) {
+__device__ __forceinline__ float token_sum(const StreamProblem& p, const float* small, size_t token, bool write, float (&h)[NP][C]) {
   const int streams = S ? S : p.streams;
   const float *mix = small, *gain = small + streams * streams, *read = gain + streams;
   const float* xr = p.x + token * p.x_token;
@@ -132,7 +131,13 @@ __device__ __forceinline__ void token_norm(const StreamProblem& p, const float* 
       for (int i = 0; i < C; ++i) ss = fmaf(h[k][i], h[k][i], ss);
     }
   }
-  const float inv = 1.0f / sqrtf(block_sum(ss, scratch) / (float)p.width + p.eps);
+  return ss;
+}
+
+// u to h, in place, from the block's sum of squares.
+template <int C, int NP>
+__device__ __forceinline__ void token_norm(const StreamProblem& p, float ss, float (&h)[NP][C]) {
+  const float inv = 1.0f / sqrtf(ss / (float)p.width + p.eps);
 #pragma unroll
   for (int k = 0; k < NP; ++k) {
     const int c = (threadIdx.x + k * blockDim.x) * C;
@@ -143,6 +148,26 @@ __device__ __forceinline__ void token_norm(const StreamProblem& p, const float* 
       for (int i = 0; i < C; ++i) h[k][i] = h[k][i] * inv * w[i];
     }
   }
+}
+
+// `block_sum` of two values at once, each in the order of `block_sum` (so either has the bits it would have alone).
+__device__ __forceinline__ float2 block_sum_pair(float a, float b, float2* scratch /* >= 33 */) {
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarps = blockDim.x >> 5;
+  a = warp_sum(a);
+  b = warp_sum(b);
+  __syncthreads();
+  if (lane == 0) scratch[warp] = make_float2(a, b);
+  __syncthreads();
+  if (threadIdx.x == 0) {
+    float2 total = make_float2(0.f, 0.f);
+    for (int w = 0; w < nwarps; ++w) {
+      total.x += scratch[w].x;
+      total.y += scratch[w].y;
+    }
+    scratch[32] = total;
+  }
+  __syncthreads();
+  return scratch[32];
 }
 
 // The small matrices into shared memory: they are weights, which no kernel writes, so this may run before the wait.
@@ -169,7 +194,8 @@ stream_norm_kernel(const StreamProblem p, T* __restrict__ out, const int* __rest
   pdl_wait();
   const size_t token = rows ? (size_t)rows[blockIdx.x] : (size_t)blockIdx.x;
   float h[NP][C];
-  token_norm<T, S, C, NP>(p, small, token, true, scratch, h);
+  const float ss = token_sum<T, S, C, NP>(p, small, token, true, h);
+  token_norm<C, NP>(p, block_sum(ss, scratch), h);
   T* o = out + (size_t)blockIdx.x * p.width;
 #pragma unroll
   for (int k = 0; k < NP; ++k) {
@@ -178,56 +204,63 @@ stream_norm_kernel(const StreamProblem p, T* __restrict__ out, const int* __rest
   }
 }
 
-// A block per tile of SHIFT_TOKENS tokens of one sequence (the tile lists name the sequence and the tile's first token).
+// A block per token. The token's h and the h of the token before it are made side by side: their loads are in flight
+// together and their sums meet in one reduction. Whether the token is a sequence's first of the step is looked up in cu_q.
+// The step's descriptors are older than every kernel of the step (the copy that brings them is no kernel, so nothing
+// overtakes it) and a state row is written by this kernel of an earlier step only, so both are read before the wait.
 template <typename T, int S, int C, int NP>
 __global__ void __launch_bounds__(MAX_THREADS)
 stream_norm_shift_kernel(const StreamProblem p, T* __restrict__ out, const float* __restrict__ mu, float* __restrict__ state,
-                         long state_stride, const int* __restrict__ cu_q, const int* __restrict__ state_slots,
-                         const int* __restrict__ tile_seq, const int* __restrict__ tile_q0) {
+                         long state_stride, const int* __restrict__ cu_q, const int* __restrict__ state_slots, int n_seqs) {
   __shared__ float small[MAX_STREAMS * MAX_STREAMS + 2 * MAX_STREAMS];
-  __shared__ float scratch[33];
+  __shared__ float2 scratch[33];
+  __shared__ int first_of;      // the sequence that starts here, or -1
   pdl_launch_dependents();
+  const size_t token = blockIdx.x;
+  if (threadIdx.x == 0) first_of = -1;
+  __syncthreads();
+  for (int i = threadIdx.x; i < n_seqs; i += blockDim.x)
+    if (cu_q[i] == (int)token) first_of = i;      // no sequence of a step is empty: at most one
   load_small(p, small);
-  pdl_wait();
-  const int seq = tile_seq[blockIdx.x], at = tile_q0[blockIdx.x];
-  const size_t row0 = (size_t)cu_q[seq];
-  const int length = cu_q[seq + 1] - (int)row0, n = min(SHIFT_TOKENS, length - at);
-  if (n <= 0) return;
-  float* row = state + (size_t)state_slots[seq] * state_stride;
+  const int seq = first_of;
   float before[NP][C], h[NP][C];
-  if (at == 0) {
+  float* row = nullptr;
+  if (seq >= 0) {
+    row = state + (size_t)state_slots[seq] * state_stride;
 #pragma unroll
     for (int k = 0; k < NP; ++k) {
       const int c = (threadIdx.x + k * blockDim.x) * C;
       if (c < p.width) Channels<float, C>::load(row + c, before[k]);
     }
   }
-  // the token before the tile (not with the state row in its place), the tile's own, and, for the state row of a sequence
-  // that goes on in other blocks, its last token
-  const int end = at == 0 && length > n ? n + 1 : n;
-  for (int j = at > 0 ? -1 : 0; j < end; ++j) {
-    const bool own = j >= 0 && j < n;
-    const size_t token = row0 + (j < n ? at + j : length - 1);
-    token_norm<T, S, C, NP>(p, small, token, own, scratch, h);
-#pragma unroll
-    for (int k = 0; k < NP; ++k) {
-      const int c = (threadIdx.x + k * blockDim.x) * C;
-      if (own && c < p.width) {
-        float m[C], v[C];
-        Channels<float, C>::load(mu + c, m);
-#pragma unroll
-        for (int i = 0; i < C; ++i) v[i] = fmaf(before[k][i] - h[k][i], m[i], h[k][i]);
-        Channels<T, C>::store(out + token * p.width + c, v);
-      }
-#pragma unroll
-      for (int i = 0; i < C; ++i) before[k][i] = h[k][i];
-    }
-  }
-  if (at > 0) return;
+  pdl_wait();
+  float ss_before = 0.f;
+  if (!row) ss_before = token_sum<T, S, C, NP>(p, small, token - 1, false, before);
+  const float ss = token_sum<T, S, C, NP>(p, small, token, true, h);
+  const float2 sums = block_sum_pair(ss, ss_before, scratch);
+  token_norm<C, NP>(p, sums.x, h);
+  if (!row) token_norm<C, NP>(p, sums.y, before);
 #pragma unroll
   for (int k = 0; k < NP; ++k) {
     const int c = (threadIdx.x + k * blockDim.x) * C;
-    if (c < p.width) Channels<float, C>::store(row + c, before[k]);
+    if (c < p.width) {
+      float m[C], v[C];
+      Channels<float, C>::load(mu + c, m);
+#pragma unroll
+      for (int i = 0; i < C; ++i) v[i] = fmaf(before[k][i] - h[k][i], m[i], h[k][i]);
+      Channels<T, C>::store(out + token * p.width + c, v);
+    }
+  }
+  if (!row) return;
+  const size_t end = (size_t)cu_q[seq + 1] - 1;
+  if (end != token) {     // the sequence goes on in other blocks: its last token's h once more, for the state row
+    const float last = token_sum<T, S, C, NP>(p, small, end, false, h);
+    token_norm<C, NP>(p, block_sum_pair(last, 0.f, scratch).x, h);
+  }
+#pragma unroll
+  for (int k = 0; k < NP; ++k) {
+    const int c = (threadIdx.x + k * blockDim.x) * C;
+    if (c < p.width) Channels<float, C>::store(row + c, h[k]);
   }
 }
 
@@ -235,14 +268,15 @@ struct ShiftArguments {
   const float* mu;
   float* state;
   long state_stride;
-  const int *cu_q, *state_slots, *tile_seq, *tile_q0;
+  const int *cu_q, *state_slots;
+  int n_seqs;
 };
 
 template <typename T, int S, int C, int NP>
 int launch_streams(const StreamProblem& p, void* out, const int* rows, int blocks, int threads, const ShiftArguments& sh, cudaStream_t stream) {
   if (sh.mu)
     lb_launch(stream_norm_shift_kernel<T, S, C, NP>, blocks, threads, 0, stream, p, (T*)out, sh.mu, sh.state, sh.state_stride, sh.cu_q,
-              sh.state_slots, sh.tile_seq, sh.tile_q0);
+              sh.state_slots, sh.n_seqs);
   else
     lb_launch(stream_norm_kernel<T, S, C, NP>, blocks, threads, 0, stream, p, (T*)out, rows);
   return lb_last_error();
@@ -257,33 +291,35 @@ int dispatch_streams(const StreamProblem& p, void* out, const int* rows, int blo
   }
   const int pieces = p.width / 4;
   if (pieces > 4 * MAX_THREADS) return LB_ERR_SIZE;
-  const int threads = pieces <= 256 ? 128 : (pieces <= 1024 ? 256 : MAX_THREADS);
+  const int threads = pieces <= 256 ? 128 : (pieces <= 512 ? 256 : MAX_THREADS);
+  const bool two = pieces <= 2 * threads;         // pieces a thread: at most two, or at most four
   switch (p.streams) {
-    case 2: return launch_streams<T, 2, 4, 4>(p, out, rows, blocks, threads, sh, stream);
-    case 4: return launch_streams<T, 4, 4, 4>(p, out, rows, blocks, threads, sh, stream);
+    case 2: return two ? launch_streams<T, 2, 4, 2>(p, out, rows, blocks, threads, sh, stream)
+                       : launch_streams<T, 2, 4, 4>(p, out, rows, blocks, threads, sh, stream);
+    case 4: return two ? launch_streams<T, 4, 4, 2>(p, out, rows, blocks, threads, sh, stream)
+                       : launch_streams<T, 4, 4, 4>(p, out, rows, blocks, threads, sh, stream);
     default: return launch_streams<T, 0, 4, 4>(p, out, rows, blocks, threads, sh, stream);
   }
 }
 }  // namespace
 
-LB_EXPORT int lb_stream_shift_tokens() { return SHIFT_TOKENS; }
 LB_EXPORT int lb_stream_max() { return MAX_STREAMS; }
 
 // x float [tokens, streams, width] by strides; y [tokens, width] of `dtype` or null (then mix and gain are null too);
 // mix float [streams, streams] ([from, to]), gain, read float [streams] (read null: ones); x_out float [tokens, streams,
 // width] or null, never the buffer of x; out [blocks, width] of `dtype`. mu null: a block per token, or per entry of
-// `rows` (then x_out is null). mu float [width]: the shifted form, `blocks` tiles, state rows of `state_stride` floats.
+// `rows` (then x_out is null). mu float [width]: the shifted form, `blocks` tokens in `n_seqs` sequences (cu_q [n_seqs + 1]:
+// their first tokens), a state row of `state_stride` floats per slot.
 LB_EXPORT int lb_stream_norm(int dtype, const float* x, long x_token, long x_stream, const void* y, const float* mix,
                              const float* gain, const float* read, float* x_out, const float* weight, float eps, void* out,
                              const int* rows, int blocks, int width, int streams, const float* mu, float* state,
-                             long state_stride, const int* cu_q, const int* state_slots, const int* tile_seq,
-                             const int* tile_q0, cudaStream_t stream) {
+                             long state_stride, const int* cu_q, const int* state_slots, int n_seqs, cudaStream_t stream) {
   if (blocks <= 0) return 0;
   if (width <= 0 || streams < 1 || streams > MAX_STREAMS || !x || !weight || !out || (y && (!mix || !gain)) || (rows && x_out) ||
-      (x_out && x_out == x) || (mu && (rows || !state || !cu_q || !state_slots || !tile_seq || !tile_q0)))
+      (x_out && x_out == x) || (mu && (rows || !state || !cu_q || !state_slots || n_seqs < 1)))
     return LB_ERR_SIZE;
   const StreamProblem p{x, x_token, x_stream, y, mix, gain, read, x_out, weight, eps, width, streams};
-  const ShiftArguments sh{mu, state, state_stride, cu_q, state_slots, tile_seq, tile_q0};
+  const ShiftArguments sh{mu, state, state_stride, cu_q, state_slots, n_seqs};
   const bool vec = width % 4 == 0 && x_token % 4 == 0 && x_stream % 4 == 0 && state_stride % 4 == 0 &&
                    ((uintptr_t)x | (uintptr_t)y | (uintptr_t)x_out | (uintptr_t)weight | (uintptr_t)out | (uintptr_t)mu |
                     (uintptr_t)state) % 16 == 0;

@@ -655,12 +655,6 @@ def gemm_tcgen05_grouped(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, ti
 
 
 # ------------------------------------------------------------------ several residual streams
-def stream_shift_tokens() -> int:
-    lib = build.load("streams")
-    lib.lb_stream_shift_tokens.restype = c_int
-    return lib.lb_stream_shift_tokens()
-
-
 def stream_norm(x: torch.Tensor, update: tuple | None, read: torch.Tensor | None, weight: torch.Tensor, eps: float,
                 out: torch.Tensor, x_out: torch.Tensor | None = None, rows: torch.Tensor | None = None,
                 shift: tuple | None = None) -> torch.Tensor:
@@ -697,21 +691,18 @@ def stream_norm(x: torch.Tensor, update: tuple | None, read: torch.Tensor | None
             raise ValueError("stream_norm: x_out is another [tokens, streams, width] buffer than x, and has no picked rows")
     if rows is not None:
         _need(rows, torch.int32, "rows")
-    mu = state = tiles = batch = None
+    mu = state = batch = None
     if shift is not None:
         mu, state, batch = shift
         _need(mu, torch.float32, "mu"); _need(state, torch.float32, "state")
         if mu.numel() != width or state.dim() != 2 or state.shape[1] < width or rows is not None or batch.n_tokens != tokens:
             raise ValueError("stream_norm: the shift is mu [width], state [slots, >= width] and this batch, without picked rows")
-        tiles = batch.tiles[stream_shift_tokens()]
-        blocks = tiles.count
     fn = _fn("streams", "lb_stream_norm", [c_int, c_void_p, c_long, c_long] + [c_void_p] * 6 + [c_float, c_void_p, c_void_p, c_int, c_int, c_int,
-                                           c_void_p, c_void_p, c_long] + [c_void_p] * 5)
+                                           c_void_p, c_void_p, c_long, c_void_p, c_void_p, c_int, c_void_p])
     _check(fn(dtype_code(out.dtype), _ptr(x), x.stride(0), x.stride(1), _ptr(y), _ptr(mix), _ptr(gain), _ptr(read), _ptr(x_out),
               _ptr(weight), float(eps), _ptr(out), _ptr(rows), blocks, width, streams, _ptr(mu), _ptr(state),
               state.stride(0) if state is not None else 0, _ptr(batch.cu_q if batch is not None else None),
-              _ptr(batch.state_slots if batch is not None else None), _ptr(tiles.tile_seq if tiles else None),
-              _ptr(tiles.tile_q0 if tiles else None), _stream()), "stream_norm")
+              _ptr(batch.state_slots if batch is not None else None), batch.n_seqs if batch is not None else 0, _stream()), "stream_norm")
     return out
 
 

@@ -320,9 +320,6 @@ class HyperConnectedBlock(Part):
     def kernel_libraries(self, dtype):
         return ("streams",)
 
-    def tile_sizes(self, dtype):
-        return (ops.stream_shift_tokens(),) if self.shift_name else ()
-
     def forward(self, x, delta, batch, cache, extra=None):
         if extra is not None or x.dim() != 3:
             raise ValueError("hyper_connected: the residual streams are [tokens, streams, hidden], and nothing else is added to them")
