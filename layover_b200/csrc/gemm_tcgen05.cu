@@ -944,6 +944,12 @@ struct Problem {
   int n_counters;
 };
 
+// A left-over round of few K blocks ends sooner whole than its tiles' partial sums meet (2,048 tokens, 3,072 outputs, 96
+// tiles of a pair: 24 -> 18 us at K = 768, 28 -> 24 at 1,536, 31 -> 29 at 2,048); longer ones are split.
+static inline bool short_left_over(const Schedule& sch, const Problem& pb) {
+  return sch.full > 0 && sch.total_kb <= 32 && pb.max_splits <= 0;
+}
+
 template <int BN, bool SWAP, typename OutT, int EPI = 0>
 int launch(const CUtensorMap& map_a, const CUtensorMap& map_b, void* C, long ldc, const Problem& pb, bool vector_ok,
            cudaStream_t stream, const int* tile_b_rows = nullptr, LbClip clip = LbClip{}) {
@@ -991,6 +997,7 @@ int launch(const CUtensorMap& map_a, const CUtensorMap& map_b, void* C, long ldc
     if (splits > cap) splits = cap;
     if (splits > sch.total_kb / 4) splits = sch.total_kb / 4;       // at least four K blocks per split
     if (splits > slots / sch.rem) splits = slots / sch.rem;
+    if (!SWAP && short_left_over(sch, pb)) splits = 1;
     const long per_split = (long)sch.rem * BN * BM;
     if (splits > 1 && per_split * splits > pb.scratch_floats) splits = (int)(pb.scratch_floats / per_split);
     if (splits > 1 && 2 * sch.rem > pb.n_counters) splits = 1;
@@ -1067,6 +1074,7 @@ int launch_pair(const CUtensorMap& map_a, const CUtensorMap& map_b, void* C, lon
     int splits = slots / sch.rem;
     if (splits > cap) splits = cap;
     if (splits > sch.total_kb / 4) splits = sch.total_kb / 4;       // at least four K blocks per split
+    if (short_left_over(sch, pb)) splits = 1;
     const long per_split = (long)sch.rem * 2 * BN * BM;              // each block of a pair has a partial tile
     if (splits > 1 && per_split * splits > pb.scratch_floats) splits = (int)(pb.scratch_floats / per_split);
     if (splits > 1 && 4 * sch.rem > pb.n_counters) splits = 1;

@@ -124,14 +124,22 @@ heads_linear_kernel(const TA* __restrict__ a, long a_row, long a_head, const T* 
       Elem<T>::store(out + (size_t)t * out_row + (size_t)h * out_head + n, v);
     }
   }
-  if (tail.room > 0 && blockIdx.y == 0) {
-    for (int i = threadIdx.x; i < HL_TOKENS * tail.room; i += 128) {
-      const int r = i / tail.room, c = i - r * tail.room, t = t0 + r;
+  if (tail.room > 0) {      // shared out over the blocks of a head's outputs; a thread turns both channels of a pair
+    const int pairs = (tail.room + 1) >> 1, half = tail.rot >> 1;
+    for (int i = blockIdx.y * 128 + threadIdx.x; i < HL_TOKENS * pairs; i += gridDim.y * 128) {
+      const int r = i / pairs, f = i - r * pairs, t = t0 + r;
       if (t >= tokens) break;
-      float v = 0.f;
-      if (c < tail.rot)
-        v = turned_channel(a + (size_t)t * a_row + (size_t)h * a_head + k_dim, tail.table + (size_t)t * tail.rot, tail.rot >> 1, c);
-      Elem<T>::store(out + (size_t)t * out_row + (size_t)h * out_head + n_out + c, v);
+      float u = 0.f, v = 0.f;
+      if (f < half) {
+        const TA* part = a + (size_t)t * a_row + (size_t)h * a_head + k_dim + 2 * f;
+        const float x = Elem<TA>::load(part), y = Elem<TA>::load(part + 1);
+        const float co = tail.table[(size_t)t * tail.rot + f], si = tail.table[(size_t)t * tail.rot + half + f];
+        u = x * co - y * si;
+        v = y * co + x * si;
+      }
+      T* dst = out + (size_t)t * out_row + (size_t)h * out_head + n_out + 2 * f;
+      Elem<T>::store(dst, u);
+      if (2 * f + 1 < tail.room) Elem<T>::store(dst + 1, v);
     }
   }
 }
