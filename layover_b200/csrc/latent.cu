@@ -21,8 +21,8 @@ __device__ __forceinline__ float turned_channel(const TA* part, const float* cs,
   return (c & 1) ? v * co + u * si : u * co - v * si;
 }
 
-// One block per token over its 32-bit projection row. The row holds [latent: rank | rotated key part: rot] at `dkv_off`:
-// c = latent * rsqrt(mean(latent^2) + eps) * norm_w goes to channels [0, rank) of the token's cache row, the rotated key
+// One block per token and latent over the token's 32-bit projection row. The row holds [latent: rank | rotated key part:
+// rot] at `dkv_off`: c = latent * rsqrt(mean(latent^2) + eps) * norm_w goes to channels [0, rank) of the token's cache row, the rotated key
 // part to [rank, rank + rot), zeros up to `room`. With `cq_rank` > 0 the row also holds the latent of the queries at
 // `cq_off`; it is normed likewise with `cq_norm_w` and left in cq_out [T, cq_rank] for the product that follows.
 template <typename T>
@@ -35,7 +35,7 @@ __global__ void latent_rows_kernel(const float* __restrict__ proj, long row_stri
   pdl_wait();
   const int t = blockIdx.x, half = rot >> 1;
   const float* row = proj + (size_t)t * row_stride;
-  if (dkv_off >= 0) {
+  if (dkv_off >= 0 && blockIdx.y == 0) {
     const float* cs = table + (size_t)t * 2 * half;
     const float* latent = row + dkv_off;
     float ss = 0.f;
@@ -50,7 +50,7 @@ __global__ void latent_rows_kernel(const float* __restrict__ proj, long row_stri
       Elem<T>::store(dst + c, v);
     }
   }
-  if (cq_rank > 0) {
+  if (cq_rank > 0 && blockIdx.y == gridDim.y - 1) {
     const float* latent = row + cq_off;
     float ss = 0.f;
     for (int c = threadIdx.x; c < cq_rank; c += blockDim.x) ss += latent[c] * latent[c];
@@ -152,11 +152,12 @@ LB_EXPORT int lb_latent_rows(int dtype, const float* proj, long row_stride, int 
   if (rot < 0 || rot % 2 || cq_rank < 0 || (cq_rank > 0 && (cq_off < 0 || !cq_norm_w || !cq_out)) || (dkv_off < 0 && cq_rank == 0) ||
       (dkv_off >= 0 && (rank <= 0 || room < rank + rot || page_tokens <= 0 || !table || !norm_w || !slot_map || !k_pool)))
     return LB_ERR_SIZE;
+  const dim3 grid(tokens, dkv_off >= 0 && cq_rank > 0 ? 2 : 1);
   if (dtype == LB_F32)
-    lb_launch(latent_rows_kernel<float>, tokens, 128, 0, stream, proj, row_stride, dkv_off, norm_w, eps, table, slot_map,
+    lb_launch(latent_rows_kernel<float>, grid, 128, 0, stream, proj, row_stride, dkv_off, norm_w, eps, table, slot_map,
               (float*)k_pool, rot, rank, room, page_tokens, cq_off, cq_rank, cq_norm_w, (float*)cq_out);
   else if (dtype == LB_BF16)
-    lb_launch(latent_rows_kernel<bf16>, tokens, 128, 0, stream, proj, row_stride, dkv_off, norm_w, eps, table, slot_map,
+    lb_launch(latent_rows_kernel<bf16>, grid, 128, 0, stream, proj, row_stride, dkv_off, norm_w, eps, table, slot_map,
               (bf16*)k_pool, rot, rank, room, page_tokens, cq_off, cq_rank, cq_norm_w, (bf16*)cq_out);
   else
     return LB_ERR_DTYPE;
