@@ -3,8 +3,8 @@
 Mimitar is a decoder with `streams` residual streams instead of one (hyper-connections: every sub-layer reads a weighted
 sum of them and all are mixed anew when its output joins, times `residual_mult`) whose layers are listed one by one. Every
 layer norms what a sub-layer reads (weights stored around zero), and what a mixer reads is first moved towards what it read
-one token before (a token shift). A layer with `weights_of` = j has no tensors of its own: it runs with layer j's, with a
-cache and a state of its own.
+one token before (a token shift). An entry with `weights_of` = j stores nothing: layer j's tensors run once more there,
+over other pages and another state.
 
 Kinds of layers (`type`):
 
