@@ -73,7 +73,7 @@ struct RotatedTail {
 };
 
 template <typename TA, typename T, int TPT>
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(128, 7)
 heads_linear_kernel(const TA* __restrict__ a, long a_row, long a_head, const T* __restrict__ w, T* __restrict__ out,
                     long out_row, long out_head, const float* __restrict__ gate, long gate_row, int gate_head, int gate_n,
                     int tokens, int n_out, int k_dim, const RotatedTail tail) {
